@@ -19,11 +19,13 @@ extern "C" {
 #define WF_SEQ_SSD 3               /* state-space recurrence with one scalar decay per head (short convolution, gated grouped norm) */
 #define WF_SEQ_MINGRU 4            /* element-wise gated recurrence: gate and candidate read only the current token */
 #define WF_SEQ_MLSTM 5             /* matrix memory with exponential input gate, sigmoid forget gate and a running maximum of the log gates */
+#define WF_SEQ_GLA 6               /* gated linear attention: matrix state per head, one decay per key channel, no write correction */
 
 /* how a layer wraps its sublayers */
 #define WF_SEQ_BLOCK_SANDWICH 0    /* x += norm_b(sub(conv(norm_a(x)))): grouped norms before and after, input convolution with carried tail */
 #define WF_SEQ_BLOCK_POST 1        /* x += residual_mult * gain * rms(sub(x)): the sublayer reads the stream, ONE gain per norm */
-#define WF_SEQ_BLOCK_PARALLEL 2    /* x += mixer(norm1(x)) + ff(norm2(x)): both branches read the same stream, each behind its own weighted norm */
+#define WF_SEQ_BLOCK_PARALLEL 2    /* x += mixer(norm1(x)) + ff(norm2(x)): both branches read the same stream, each behind its own weighted norm
+                                    * (one norm for both with one_norm; either branch times a sigmoid gate with branch_gates) */
 
 /* feed-forward kinds (wf_seq_layer.has_ff) and gated activations (ff_act) */
 #define WF_SEQ_FF_NONE 0
@@ -113,6 +115,19 @@ typedef struct wf_seq_layer {
      * divided by its root mean square, times mix.norm [heads * vdim], times sigmoid(W_g x), then W_o.  Tensors mix.q, mix.k, mix.v, mix.g,
      * mix.i, mix.i.b, mix.f, mix.f.b, mix.norm, mix.o. */
     float gate_cap;
+    /* grouped-query attention, further.  dist_log = 1: score -= r1_h ln(1 + r2_h (i - j)) with learned numbers per head (tensors mix.r1,
+     * mix.r2 [heads]).  sink = 2: as for latent attention (mix.sink).  talk = 1: the heads' softmax weights are mixed before they meet the
+     * values, weight_h <- sum_g T[h, g] weight_g (tensor mix.talk [heads, heads]; the sink's share has no weight to mix); head h applies its
+     * mixed weights to the values of its own key/value head. */
+    int dist_log, talk;
+    /* paired mixers: pair_norm = 1: each mixer's output is RMS-normed over the model width with a weight vector (tensors mix.left.out,
+     * mix.right.out) before mix_scale and pair_scale combine them. */
+    int pair_norm;
+    /* WF_SEQ_GLA: heads of key size dim and value size vdim.  q = W_q x * dim^-1/2, k, v; decay per head and key channel
+     * a = sigmoid(W_a2 (W_a1 x) + b)^(1 / decay_tau) (W_a1 has decay_rank rows); S <- diag(a) S + k v^T, o = S^T q; each head's o divided by
+     * its root mean square, times mix.norm [vdim], times silu(W_g x), then W_o.  Tensors mix.q, mix.k, mix.v, mix.g, mix.a1, mix.a2, mix.a2.b,
+     * mix.norm, mix.o. */
+    float decay_tau;
 } wf_seq_layer;
 
 typedef struct wf_seq_config {
@@ -125,13 +140,20 @@ typedef struct wf_seq_config {
     int max_step_tokens;           /* most tokens in one step */
     int block_form;                /* WF_SEQ_BLOCK_* */
     float residual_mult;           /* WF_SEQ_BLOCK_POST */
-    int pos_embed;                 /* 1: a sinusoidal position vector is added to the embedding (entry 2i sin, 2i + 1 cos of p * pos_base^(-2i / width)) */
+    int pos_embed;                 /* 1: a sinusoidal position vector is added to the embedding (entry 2i sin, 2i + 1 cos of p * pos_base^(-2i / width));
+                                    * 2: a learned one (tensor 'pos' [max_positions, width]), not scaled with the embedding */
     float pos_base;
     int n_extra;                   /* mixer descriptors behind the n_layers layer entries (the second mixers of paired layers) */
     float embed_scale;             /* the embedding row is multiplied by this (0 is read as 1) */
     int norm_weights;              /* WF_SEQ_BLOCK_POST: 1 = the norms have weight vectors of the width instead of a single gain */
     int tied_head;                 /* 1: logits are products with the embedding table itself; there is no 'head' tensor */
     float norm_offset;             /* added to every stored weight of the layer norms and the final norm (1: weights stored around zero) */
+    int layer_norm;                /* WF_SEQ_BLOCK_PARALLEL: 1 = the norms take the mean off and have biases (tensors '<norm>.b') */
+    int one_norm;                  /* WF_SEQ_BLOCK_PARALLEL: 1 = both branches read norm1's output (attention and WF_SEQ_GLA mixers) */
+    int branch_gates;              /* with one_norm: a branch's result times sigmoid(W h + b), h the norm's output, per element (tensors 'l<i>.rg1',
+                                    * 'l<i>.rg1.b' for the mixer, 'l<i>.rg2', 'l<i>.rg2.b' for the feed-forward) */
+    int max_positions;             /* pos_embed = 2: rows of the position table; no sequence grows longer */
+    float logit_softcap;           /* > 0: logits <- cap * tanh(logits / cap) */
 } wf_seq_config;
 
 typedef struct wf_seq_engine wf_seq_engine;
@@ -172,7 +194,7 @@ int wf_seq_launches_last_step(const wf_seq_engine* e);
  * [n, width]) through the same kernels, caches and state as wf_seq_step, and returns that part's float output [n, width]:
  * 0 first norm, 1 input convolution of the mixer (carried state), 2 the mixer, 3 the feed-forward, 4 input convolution of the
  * feed-forward (1 and 4: WF_SEQ_BLOCK_SANDWICH only; part 0 of WF_SEQ_BLOCK_POST is residual_mult * gain * rms(rows)), 5 second norm
- * (WF_SEQ_BLOCK_PARALLEL only).
+ * (WF_SEQ_BLOCK_PARALLEL with two norms only).
  * Sequence lengths advance as in a step. */
 int wf_seq_set_layer_tap(wf_seq_engine* e, float* host);
 int wf_seq_run_part(wf_seq_engine* e, int layer, int part, int nseq, const int32_t* slots, const int32_t* counts, const float* in_host,

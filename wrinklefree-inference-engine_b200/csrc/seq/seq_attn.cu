@@ -1,7 +1,8 @@
 // Grouped-query softmax attention over a paged cache of per-head keys and values.  Positions can enter through a rotation of queries and
 // keys (partial, pairs interleaved or split in halves), through a linear distance penalty per head (score -= slope_h * (i - j),
 // slope_h = 2^(-dist_exp (h + 1) / H)) or through a learned bias by distance; the visible keys are the causal ones inside a sliding window
-// and / or inside the query's own chunk of positions; scores can be capped by a tanh and the softmax denominator can carry an extra one.
+// and / or inside the query's own chunk of positions; scores can be capped by a tanh, lowered by a logarithm of the distance, and the softmax
+// denominator can carry an extra one or a learned sink per head; the heads' weights can be mixed by a matrix before they meet the values.
 // Queries, keys and values can be normalised before use (per head, with or without weights, or over the whole projection; the cache holds
 // keys and values in that form), and the output can be multiplied by a sigmoid gate computed from the layer input, per head or per element.
 // A layer may read the cache rows that an earlier layer wrote instead of projecting its own.
@@ -152,6 +153,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_attn_kernel(Batch b, GqaDim
         if (D.softcap > 0.f) sc = D.softcap * tanhf(sc / D.softcap);
         if (D.rel) { const int dist = pos - j; sc += D.rel[(size_t)(dist < D.rel_n ? dist : D.rel_n - 1) * D.H + h]; }
         sc -= slope * (float)(pos - j);
+        if (D.dist_r1) sc -= D.dist_r1[h] * log1pf(D.dist_r2[h] * (float)(pos - j));
         const float mn = fmaxf(m, sc);
         const float corr = expf(m - mn);      // m = -inf on the first key: exp(-inf) = 0
         const float p = expf(sc - mn);
@@ -173,7 +175,12 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_attn_kernel(Batch b, GqaDim
     float lg = 0.f, sc_w[GA_WARPS];
 #pragma unroll
     for (int w = 0; w < GA_WARPS; ++w) { sc_w[w] = part_m[w] == -INFINITY ? 0.f : expf(part_m[w] - mg); lg += part_l[w] * sc_w[w]; }
-    if (D.sink) lg += expf(-mg);            // the extra key: score 0, no value
+    if (D.sink) {                           // the extra key (score 0 or a learned one) has no value; its share may be the largest
+        const float ms = D.sink_h ? D.sink_h[h] : 0.f, top = fmaxf(mg, ms), f = expf(mg - top);
+        lg = lg * f + expf(ms - top);
+#pragma unroll
+        for (int w = 0; w < GA_WARPS; ++w) sc_w[w] *= f;
+    }
     const float inv_l = 1.f / lg;
     const float* grow = gate ? (D.gate_elem ? gate + ((size_t)i * D.H + h) * D.dv : gate + (size_t)i * D.H + h) : nullptr;
     for (int c = threadIdx.x; c < D.dv; c += blockDim.x) {
@@ -182,6 +189,97 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_attn_kernel(Batch b, GqaDim
         for (int w = 0; w < GA_WARPS; ++w) v += part_sum[w * D.dv + c] * sc_w[w];
         const float gm = grow ? (D.gate_elem ? grow[c] : grow[0]) : 1.f;
         out[((size_t)i * D.H + h) * D.dv + c] = from_f<T>(v * inv_l * gm);
+    }
+}
+
+// Mixed heads: head h's weights are sum_g talk[h, g] * (head g's softmax weights), so a token's heads run together, and since the mixture
+// needs normalised weights the keys are walked twice: once for every head's maximum and sum, once for weights, mixture and values.
+// One block per token; GT_KEYS keys at a time.  Scores of a tile lie in shared memory [H][GT_KEYS], their mixture beside them, the output
+// accumulators [H][dv] too (any sizes that fit: the launcher checks).
+constexpr int GT_KEYS = 32, GT_THREADS = 256;
+template <typename T>
+__global__ void __launch_bounds__(GT_THREADS) gqa_talk_attn_kernel(Batch b, GqaDims D, const T* __restrict__ qn, const float* __restrict__ gate, PagedCache pc,
+                                                                   T* __restrict__ out) {
+    extern __shared__ float sm[];
+    float* sc = sm;                                   // [H][GT_KEYS] scores, then normalised weights
+    float* mix = sc + D.H * GT_KEYS;                  // [H][GT_KEYS] mixed weights
+    float* acc = mix + D.H * GT_KEYS;                 // [H][dv]
+    float* hm = acc + D.H * D.dv;                     // [H] running maximum
+    float* hl = hm + D.H;                             // [H] running sum, then 1 / denominator
+    const int i = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = GT_THREADS / 32;
+    const int sq = b.tok_seq[i], pos = b.tok_pos[i], rep = D.H / D.G;
+    int lo = pos - D.window + 1 > 0 ? pos - D.window + 1 : 0;
+    if (D.chunk > 0) { const int c0 = pos / D.chunk * D.chunk; if (c0 > lo) lo = c0; }
+    const int32_t* bt = pc.block_table + (size_t)b.seq_slot[sq] * pc.max_blocks;
+    auto page_of = [&](int j) { return (const T*)pc.pool + (size_t)bt[j / pc.page_size] * pc.page_stride + pc.layer_off; };
+    auto scores = [&](int j0, int cnt) {              // a warp per (head, key), lanes over the dimensions
+        for (int u = warp; u < D.H * cnt; u += nw) {
+            const int h = u / cnt, k = u - h * cnt, j = j0 + k, dist = pos - j;
+            const T* kr = page_of(j) + ((size_t)(h / rep) * pc.page_size + j % pc.page_size) * D.d;
+            const T* qh = qn + ((size_t)i * D.H + h) * D.d;
+            float part = 0.f;
+            for (int c = lane; c < D.d; c += 32) part = fmaf(to_f(qh[c]), to_f(kr[c]), part);
+            float v = warp_sum(part) * D.scale;
+            if (D.softcap > 0.f) v = D.softcap * tanhf(v / D.softcap);
+            if (D.rel) v += D.rel[(size_t)(dist < D.rel_n ? dist : D.rel_n - 1) * D.H + h];
+            if (D.dist_exp > 0.f) v -= exp2f(-D.dist_exp * (float)(h + 1) / (float)D.H) * (float)dist;
+            if (D.dist_r1) v -= D.dist_r1[h] * log1pf(D.dist_r2[h] * (float)dist);
+            if (lane == 0) sc[h * GT_KEYS + k] = v;
+        }
+    };
+    for (int h = threadIdx.x; h < D.H; h += GT_THREADS) {
+        hm[h] = D.sink ? (D.sink_h ? D.sink_h[h] : 0.f) : -INFINITY;
+        hl[h] = D.sink ? 1.f : 0.f;                   // the sink opens the sum and is its own maximum so far
+    }
+    for (int e = threadIdx.x; e < D.H * D.dv; e += GT_THREADS) acc[e] = 0.f;
+    for (int j0 = lo; j0 <= pos; j0 += GT_KEYS) {
+        const int cnt = pos - j0 + 1 < GT_KEYS ? pos - j0 + 1 : GT_KEYS;
+        __syncthreads();
+        scores(j0, cnt);
+        __syncthreads();
+        for (int h = warp; h < D.H; h += nw) {
+            const float v = lane < cnt ? sc[h * GT_KEYS + lane] : -INFINITY;
+            const float mo = hm[h], mn = fmaxf(mo, warp_max(v));
+            const float ls = warp_sum(lane < cnt ? expf(v - mn) : 0.f);
+            __syncwarp();
+            if (lane == 0) { hl[h] = hl[h] * expf(mo - mn) + ls; hm[h] = mn; }
+        }
+    }
+    __syncthreads();
+    for (int h = threadIdx.x; h < D.H; h += GT_THREADS) hl[h] = 1.f / hl[h];
+    for (int j0 = lo; j0 <= pos; j0 += GT_KEYS) {
+        const int cnt = pos - j0 + 1 < GT_KEYS ? pos - j0 + 1 : GT_KEYS;
+        __syncthreads();
+        scores(j0, cnt);
+        __syncthreads();
+        for (int e = threadIdx.x; e < D.H * GT_KEYS; e += GT_THREADS) {
+            const int h = e / GT_KEYS;
+            sc[e] = e - h * GT_KEYS < cnt ? expf(sc[e] - hm[h]) * hl[h] : 0.f;
+        }
+        __syncthreads();
+        for (int e = threadIdx.x; e < D.H * GT_KEYS; e += GT_THREADS) {
+            const int h = e / GT_KEYS, k = e - h * GT_KEYS;
+            float v = 0.f;
+            for (int g = 0; g < D.H; ++g) v = fmaf(D.talk[h * D.H + g], sc[g * GT_KEYS + k], v);
+            mix[e] = v;
+        }
+        __syncthreads();
+        for (int e = threadIdx.x; e < D.H * D.dv; e += GT_THREADS) {
+            const int h = e / D.dv, c = e - h * D.dv, g = h / rep;
+            float v = acc[e];
+            for (int k = 0; k < cnt; ++k) {
+                const int j = j0 + k;
+                const size_t at = D.v_is_k ? ((size_t)g * pc.page_size + j % pc.page_size) * D.d
+                                           : (size_t)D.G * pc.page_size * D.d + ((size_t)g * pc.page_size + j % pc.page_size) * D.dv;
+                v = fmaf(mix[h * GT_KEYS + k], to_f(page_of(j)[at + c]), v);
+            }
+            acc[e] = v;
+        }
+    }
+    __syncthreads();
+    for (int e = threadIdx.x; e < D.H * D.dv; e += GT_THREADS) {
+        const float gm = gate ? (D.gate_elem ? gate[(size_t)i * D.H * D.dv + e] : gate[(size_t)i * D.H + e / D.dv]) : 1.f;
+        out[(size_t)i * D.H * D.dv + e] = from_f<T>(acc[e] * gm);
     }
 }
 
@@ -213,6 +311,18 @@ int launch_gqa_attn(int dt, const Batch& b, const GqaDims& D, const void* qn, co
     if (b.n <= 0) return WF_OK;
     if (int rc = check_dims(D)) return rc;
     if (D.H > 65535) { set_error("attention: too many heads"); return WF_ERR_UNSUPPORTED; }
+    if (D.talk) {
+        const size_t bytes = ((size_t)2 * D.H * GT_KEYS + (size_t)D.H * D.dv + 2 * D.H) * sizeof(float);
+        if (bytes > 200 * 1024) { set_error("attention: %d mixed heads of %d values exceed shared memory", D.H, D.dv); return WF_ERR_UNSUPPORTED; }
+        static DevOnce once;
+        if (once.need()) {
+            cudaFuncSetAttribute(gqa_talk_attn_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+            cudaFuncSetAttribute(gqa_talk_attn_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        }
+        if (dt == WF_BF16) gqa_talk_attn_kernel<<<b.n, GT_THREADS, bytes, s>>>(b, D, (const __nv_bfloat16*)qn, gate, pc, (__nv_bfloat16*)out);
+        else gqa_talk_attn_kernel<<<b.n, GT_THREADS, bytes, s>>>(b, D, (const float*)qn, gate, pc, (float*)out);
+        return launch_check(cudaGetLastError(), "gqa_talk_attn");
+    }
     dim3 grid(b.n, D.H);
     const size_t smem = ((size_t)GA_WARPS * D.dv + 2 * GA_WARPS) * sizeof(float);
     if (dt == WF_BF16) gqa_attn_kernel<<<grid, GA_WARPS * 32, smem, s>>>(b, D, (const __nv_bfloat16*)qn, gate, pc, (__nv_bfloat16*)out);

@@ -12,7 +12,7 @@
 //   * decode form (every sequence brings one token): the four warps share the same 16 rows and each takes 16 keys of a tile; the key
 //     range can also be cut over `splits` CTAs.  Partial (max, sum, weighted values) are merged through shared memory and, with splits,
 //     through a float workspace and a merge kernel.
-#include "seq_kernels.cuh"
+#include "seq_attn_mma.cuh"
 #include <math.h>
 #include <stdlib.h>
 
@@ -23,28 +23,6 @@ namespace {
 
 constexpr int AM_THREADS = 128;
 constexpr int AM_KT = 64;                 // keys per staged tile
-constexpr float LOG2E = 1.4426950408889634f;
-
-__device__ __forceinline__ void am_ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void am_ldsm_x4_trans(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void am_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void am_cp16(uint32_t dst, const void* src, bool valid) {
-    const int sz = valid ? 16 : 0;          // 0: the 16 bytes are zero-filled
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
-}
-__device__ __forceinline__ void am_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void am_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&v);
-}
 
 struct AmParams {
     int rp2, rp2_log;        // rows per token: the group size rounded up to a power of two
@@ -103,6 +81,11 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
         r_slope2[k] = D.dist_exp > 0.f ? exp2f(-D.dist_exp * (float)(r_head[k] + 1) / (float)D.H) * LOG2E : 0.f;
     }
     const float scale2 = D.scale * LOG2E;
+    float r_lr1[2] = {0.f, 0.f}, r_lr2[2] = {0.f, 0.f};    // logarithmic penalty of the row's head; r1 ln(x) log2 e = r1 log2(x)
+    if (EXT && D.dist_r1) {
+#pragma unroll
+        for (int k = 0; k < 2; ++k) { r_lr1[k] = D.dist_r1[r_head[k]]; r_lr2[k] = D.dist_r2[r_head[k]]; }
+    }
     const float cap2 = D.softcap > 0.f ? 2.f / D.softcap : 0.f;
     // first and last position among the rows of this warp that exist
     const int wpos_min = pos0 + (row_base >> ap.rp2_log);
@@ -233,7 +216,9 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
                     // score to a few 1e-6 of the cap, well inside what the bf16 operands of the product leave
                     if (D.softcap > 0.f) v = D.softcap * (1.f - __fdividef(2.f, __expf(v * cap2) + 1.f));
                     if (D.rel) { const int dd = max(0, min(dist, D.rel_n - 1)); v += __ldg(D.rel + dd * D.H + r_head[k]); }
-                    v = vis ? fmaf(v, LOG2E, -r_slope2[k] * (float)dist) : -INFINITY;
+                    float pen = r_slope2[k] * (float)dist;
+                    if (D.dist_r1) pen = fmaf(r_lr1[k], __log2f(fmaf(r_lr2[k], (float)dist, 1.f)), pen);
+                    v = vis ? fmaf(v, LOG2E, -pen) : -INFINITY;
                     s[j][e] = v;
                     mx[k] = fmaxf(mx[k], v);
                 }
@@ -321,8 +306,7 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             if (!r_ok[k]) continue;
-            const float lsum = D.sink ? l_run[k] + exp2f(-m_run[k]) : l_run[k];      // the extra key: score 0, no value
-            const float mul = (gate && !D.gate_elem ? gate[(size_t)r_tok[k] * D.H + r_head[k]] : 1.f) / lsum;
+            const float mul = (gate && !D.gate_elem ? gate[(size_t)r_tok[k] * D.H + r_head[k]] : 1.f) * am_inv_sum(D, r_head[k], m_run[k], l_run[k]);
             __nv_bfloat16* dst = out + ((size_t)r_tok[k] * D.H + r_head[k]) * D.dv;
             const float* ge = gate && D.gate_elem ? gate + ((size_t)r_tok[k] * D.H + r_head[k]) * D.dv : nullptr;
 #pragma unroll
@@ -369,8 +353,7 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
             }
             if (lane == 0) { dst[D.dv] = mg; dst[D.dv + 1] = lg; }
         } else {
-            if (D.sink) lg += exp2f(-mg);
-            const float mul = (gate && !D.gate_elem ? gate[(size_t)tok * D.H + head] : 1.f) / lg;
+            const float mul = (gate && !D.gate_elem ? gate[(size_t)tok * D.H + head] : 1.f) * am_inv_sum(D, head, mg, lg);
             const float* ge = gate && D.gate_elem ? gate + ((size_t)tok * D.H + head) * D.dv : nullptr;
             for (int c = lane; c < D.dv; c += 32) {
                 float v = 0.f;
@@ -383,8 +366,8 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
 }
 
 // one warp per (token, head): merge the key splits' partial results (maxima in units of log 2), apply the gate
-__global__ void gqa_attn_merge_kernel(int rows, int splits, int dv, const float* __restrict__ part, const float* __restrict__ gate, __nv_bfloat16* __restrict__ out,
-                                      int sink, int gate_elem) {
+__global__ void gqa_attn_merge_kernel(GqaDims D, int rows, int splits, const float* __restrict__ part, const float* __restrict__ gate, __nv_bfloat16* __restrict__ out) {
+    const int dv = D.dv, gate_elem = D.gate_elem;
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= rows) return;
     const float* p = part + (size_t)row * splits * (dv + 2);
@@ -392,8 +375,7 @@ __global__ void gqa_attn_merge_kernel(int rows, int splits, int dv, const float*
     for (int z = 0; z < splits; ++z) mg = fmaxf(mg, p[(size_t)z * (dv + 2) + dv]);
     float lg = 0.f;
     for (int z = 0; z < splits; ++z) { const float m = p[(size_t)z * (dv + 2) + dv]; lg += m == -INFINITY ? 0.f : p[(size_t)z * (dv + 2) + dv + 1] * exp2f(m - mg); }
-    if (sink) lg += exp2f(-mg);
-    const float mul = (gate && !gate_elem ? gate[row] : 1.f) / lg;
+    const float mul = (gate && !gate_elem ? gate[row] : 1.f) * am_inv_sum(D, row % D.H, mg, lg);
     for (int c = lane; c < dv; c += 32) {
         float v = 0.f;
         for (int z = 0; z < splits; ++z) { const float m = p[(size_t)z * (dv + 2) + dv]; if (m != -INFINITY) v += p[(size_t)z * (dv + 2) + c] * exp2f(m - mg); }
@@ -419,7 +401,7 @@ int am_launch(const Batch& b, const GqaDims& D, const void* qn, const float* gat
 template <bool DECODE, int NSTAGE>
 int am_dispatch(const Batch& b, const GqaDims& D, const void* qn, const float* gate, const PagedCache& pc, void* out, const AmParams& ap, int tiles, cudaStream_t s) {
     const bool k64 = D.d <= 64, v64 = D.dv <= 64;
-    if (D.softcap > 0.f || D.rel) {
+    if (D.softcap > 0.f || D.rel || D.dist_r1) {
         if (k64 && v64) return am_launch<64, 64, DECODE, NSTAGE, true>(b, D, qn, gate, pc, out, ap, tiles, s);
         if (k64) return am_launch<64, 128, DECODE, NSTAGE, true>(b, D, qn, gate, pc, out, ap, tiles, s);
         if (v64) return am_launch<128, 64, DECODE, NSTAGE, true>(b, D, qn, gate, pc, out, ap, tiles, s);
@@ -441,7 +423,7 @@ bool gqa_attn_mma_usable(const GqaDims& D, const PagedCache& pc) {
            ((long long)pc.page_size * D.d) % 8 == 0 && D.G <= 65535;
 }
 
-bool gqa_attn_mma_takes(const GqaDims& D) { return D.chunk >= 0 && D.softcap >= 0.f; }
+bool gqa_attn_mma_takes(const GqaDims& D) { return D.chunk >= 0 && D.softcap >= 0.f && !D.talk; }
 
 size_t gqa_attn_mma_workspace(int rows, int splits, int dv) { return (size_t)rows * splits * (dv + 2) * sizeof(float); }
 
@@ -466,7 +448,7 @@ int launch_gqa_attn_mma(const Batch& b, const GqaDims& D, const void* qn, const 
                      : (g_decode_stages == 3 ? am_dispatch<true, 3>(b, D, qn, gate, pc, out, ap, tiles, s) : am_dispatch<true, 2>(b, D, qn, gate, pc, out, ap, tiles, s));
     if (rc || ap.splits == 1) return rc;
     const int rows = b.n * D.H;
-    gqa_attn_merge_kernel<<<(rows + 3) / 4, 128, 0, s>>>(rows, ap.splits, D.dv, workspace, gate, (__nv_bfloat16*)out, D.sink, D.gate_elem);
+    gqa_attn_merge_kernel<<<(rows + 3) / 4, 128, 0, s>>>(D, rows, ap.splits, workspace, gate, (__nv_bfloat16*)out);
     return launch_check(cudaGetLastError(), "gqa_attn_merge");
 }
 

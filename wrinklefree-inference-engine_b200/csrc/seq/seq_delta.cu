@@ -1,6 +1,7 @@
 // Gated delta rule: a per-head matrix state S [d, dv] in float that every token first decays (one factor per head, or one per head and key
 // row), then corrects along its key (u = beta (v - S^T k), S += k u^T) and finally reads with its query (o = S^T q).  The same kernel
-// without the correction (u = beta v) is the state-space recurrence S = a S + dt B x^T, y = S^T C with k = B, q = C, v = x, beta = dt.
+// without the correction (u = beta v) is the state-space recurrence S = a S + dt B x^T, y = S^T C with k = B, q = C, v = x, beta = dt, and,
+// with one decay per key row and beta = 1, gated linear attention S = diag(a) S + k v^T.
 // The state is carried per sequence slot across steps.
 #include "seq_kernels.cuh"
 
@@ -117,7 +118,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDi
         const size_t entry = ((size_t)(start / sa.chunk + sq + c) * D.H + h) * D.d * dvs;
         S = sa.pass == 1 ? nullptr : sa.start + entry;
         S_out = sa.pass == 1 ? sa.local + entry : nullptr;
-        if (sa.pass == 1 && tid == 0 && blockIdx.z == 0) {                                   // the chunk's decay product (one decay per head)
+        if (!VEC && sa.pass == 1 && tid == 0 && blockIdx.z == 0) {                           // the chunk's decay product (one decay per head)
             float pr = 1.f;
             const int t1 = len - c * sa.chunk < sa.chunk ? len - c * sa.chunk : sa.chunk;
             for (int t = 0; t < t1; ++t) pr *= decay[(size_t)(start + c * sa.chunk + t) * D.H + h];
@@ -176,7 +177,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDi
             }
         }
         if (tid < tt) {
-            cp_async4(bs + tid, beta + (size_t)(start + t0 + tid) * D.H + h);
+            if (beta) cp_async4(bs + tid, beta + (size_t)(start + t0 + tid) * D.H + h); else bs[tid] = 1.f;
             if (!VEC) cp_async4(gs + tid, decay + (size_t)(start + t0 + tid) * D.H + h);
         }
         cp_async_commit();
@@ -256,7 +257,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDi
             os += __shfl_xor_sync(0xffffffffu, os, 1);
             os += __shfl_xor_sync(0xffffffffu, os, 2);
             if (DR_PARTS == 8) os += __shfl_xor_sync(0xffffffffu, os, 4);
-            if (p == 0 && col_ok) o[((size_t)(start + t0 + t) * D.H + h) * dvs + col] = os;
+            if (p == 0 && col_ok) o[((size_t)(start + t0 + t) * D.H + h) * dvs + col] = os * D.o_scale;
         }
     }
     if (!S_out) return;
@@ -267,9 +268,10 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDi
     }
 }
 
-// thread per (sequence, head, state element): chains the chunks' start states from the slot's state and leaves the end state in the slot
+// thread per (sequence, head, state element): chains the chunks' start states from the slot's state and leaves the end state in the slot.
+// prod has one entry per (chunk, head), or (d > 0) one per (chunk, head, key row) of dd / d state columns each
 __global__ void scan_prefix_kernel(Batch b, int H, int dd, int chunk, float* __restrict__ state, size_t slot_stride, const float* __restrict__ local,
-                                   float* __restrict__ startws, const float* __restrict__ prod) {
+                                   float* __restrict__ startws, const float* __restrict__ prod, int d) {
     const int sq = blockIdx.x, h = blockIdx.y, e = blockIdx.z * blockDim.x + threadIdx.x;
     if (e >= dd) return;
     const int len = b.seq_len[sq], nc = (len + chunk - 1) / chunk, base = b.seq_start[sq] / chunk + sq;
@@ -278,9 +280,54 @@ __global__ void scan_prefix_kernel(Batch b, int H, int dd, int chunk, float* __r
     for (int c = 0; c < nc; ++c) {
         const size_t entry = (size_t)(base + c) * H + h;
         startws[entry * dd + e] = S;
-        S = fmaf(prod[entry], S, local[entry * dd + e]);
+        S = fmaf(d > 0 ? prod[entry * d + e / (dd / d)] : prod[entry], S, local[entry * dd + e]);
     }
     *Sp = S;
+}
+
+// thread per (sequence and chunk, head and key row): the product of the chunk's decays
+__global__ void scan_decay_prod_kernel(Batch b, int nd, int chunk, int nchunks, const float* __restrict__ decay, float* __restrict__ prod) {
+    const int sq = blockIdx.x / nchunks, c = blockIdx.x - sq * nchunks, k = blockIdx.y * blockDim.x + threadIdx.x;
+    const int len = b.seq_len[sq], start = b.seq_start[sq];
+    if (k >= nd || c * chunk >= len) return;
+    const int t1 = len - c * chunk < chunk ? len - c * chunk : chunk;
+    const float* p = decay + (size_t)(start + c * chunk) * nd + k;
+    float pr = 1.f;
+#pragma unroll 8
+    for (int t = 0; t < t1; ++t) pr *= p[(size_t)t * nd];
+    prod[(size_t)(start / chunk + sq + c) * nd + k] = pr;
+}
+
+// decay of gated linear attention: a thread owns one output channel and GD_TOK tokens; the tokens' low-rank rows lie in shared memory
+constexpr int GD_TOK = 8, GD_THREADS = 128;
+template <typename T>
+__global__ void __launch_bounds__(GD_THREADS) gla_decay_kernel(int n, int rank, int nout, const float* __restrict__ a1, int ld, const T* __restrict__ a2,
+                                                               const T* __restrict__ bias, float inv_tau, float* __restrict__ decay) {
+    extern __shared__ float rows[];                  // [rank][GD_TOK]
+    const int i0 = blockIdx.x * GD_TOK, c = blockIdx.y * GD_THREADS + threadIdx.x;
+    for (int idx = threadIdx.x; idx < rank * GD_TOK; idx += GD_THREADS) {
+        const int t = idx / rank, r = idx - t * rank;
+        rows[r * GD_TOK + t] = i0 + t < n ? a1[(size_t)(i0 + t) * ld + r] : 0.f;
+    }
+    __syncthreads();
+    if (c >= nout) return;
+    float acc[GD_TOK];
+    const float bz = to_f(bias[c]);
+#pragma unroll
+    for (int t = 0; t < GD_TOK; ++t) acc[t] = bz;
+    const T* wr = a2 + (size_t)c * rank;
+#pragma unroll 4
+    for (int r = 0; r < rank; ++r) {
+        const float w = to_f(wr[r]);
+#pragma unroll
+        for (int t = 0; t < GD_TOK; ++t) acc[t] = fmaf(w, rows[r * GD_TOK + t], acc[t]);
+    }
+#pragma unroll
+    for (int t = 0; t < GD_TOK; ++t)
+        if (i0 + t < n) {
+            const float z = acc[t];                  // ln sigmoid(z) = min(z, 0) - ln(1 + exp(-|z|))
+            decay[(size_t)(i0 + t) * nout + c] = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
+        }
 }
 
 template <typename T>
@@ -347,21 +394,29 @@ int launch_delta_rule(const Batch& b, const DeltaDims& D, const float* qkv, int 
     if (D.Hk <= 0 || D.H % D.Hk) { set_error("delta: %d heads over %d key heads", D.H, D.Hk); return WF_ERR_INVALID; }
     if (D.ones_col && !D.no_delta) { set_error("delta: the all-ones column belongs to the plain recurrence"); return WF_ERR_UNSUPPORTED; }
     if (D.no_delta) {
-        if (D.vec_decay) { set_error("delta: the plain recurrence takes one decay per head"); return WF_ERR_UNSUPPORTED; }
+        auto plain = [&](const ScanArgs& sa) {
+            return D.vec_decay ? delta_rule_launch<true, false>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s, sa)
+                               : delta_rule_launch<false, false>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s, sa);
+        };
         // long portions: chunks in parallel (two short sequential passes instead of one long one)
         if (scan && scan->local && b.n != b.nseq && b.max_len >= 2 * SCAN_CHUNK && b.n / SCAN_CHUNK + b.nseq + 1 <= scan->chunks) {
             ScanArgs sa;
             sa.chunk = SCAN_CHUNK; sa.nchunks = (b.max_len + SCAN_CHUNK - 1) / SCAN_CHUNK;
             sa.local = scan->local; sa.start = scan->start; sa.prod = scan->prod;
             sa.pass = 1;
-            if (int rc = delta_rule_launch<false, false>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s, sa)) return rc;
+            if (int rc = plain(sa)) return rc;
+            if (D.vec_decay) {
+                const int nd = D.H * D.d;
+                scan_decay_prod_kernel<<<dim3(b.nseq * sa.nchunks, (nd + 127) / 128), 128, 0, s>>>(b, nd, SCAN_CHUNK, sa.nchunks, decay, scan->prod);
+                if (int rc = launch_check(cudaGetLastError(), "scan_decay_prod")) return rc;
+            }
             const int dd = D.d * (D.dv + D.ones_col);
-            scan_prefix_kernel<<<dim3(b.nseq, D.H, (dd + 255) / 256), 256, 0, s>>>(b, D.H, dd, SCAN_CHUNK, state, slot_stride, scan->local, scan->start, scan->prod);
+            scan_prefix_kernel<<<dim3(b.nseq, D.H, (dd + 255) / 256), 256, 0, s>>>(b, D.H, dd, SCAN_CHUNK, state, slot_stride, scan->local, scan->start, scan->prod, D.vec_decay ? D.d : 0);
             if (int rc = launch_check(cudaGetLastError(), "scan_prefix")) return rc;
             sa.pass = 3;
-            return delta_rule_launch<false, false>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s, sa);
+            return plain(sa);
         }
-        return delta_rule_launch<false, false>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s);
+        return plain(ScanArgs());
     }
     return D.vec_decay ? delta_rule_launch<true, true>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s)
                        : delta_rule_launch<false, true>(b, D, qkv, ld, beta, decay, state, slot_stride, o, s);
@@ -373,6 +428,16 @@ int launch_delta_post(int dt, const DeltaDims& D, int n, const float* o, const v
     if (dt == WF_BF16) delta_post_kernel<<<grid, 128, 0, s>>>(D, o, (const __nv_bfloat16*)w, eps, g, ldg, (__nv_bfloat16*)y, act);
     else delta_post_kernel<<<grid, 128, 0, s>>>(D, o, (const float*)w, eps, g, ldg, (float*)y, act);
     return launch_check(cudaGetLastError(), "delta_post");
+}
+
+int launch_gla_decay(int dt, int n, int rank, int nout, const float* a1, int ld, const void* a2, const void* bias, float tau, float* decay, cudaStream_t s) {
+    if (n <= 0) return WF_OK;
+    const size_t smem = (size_t)rank * GD_TOK * sizeof(float);
+    if (rank <= 0 || !(tau > 0.f) || smem > 48 * 1024) { set_error("gla: decay projection of rank %d, tau %g", rank, tau); return WF_ERR_UNSUPPORTED; }
+    const dim3 grid((n + GD_TOK - 1) / GD_TOK, (nout + GD_THREADS - 1) / GD_THREADS);
+    if (dt == WF_BF16) gla_decay_kernel<<<grid, GD_THREADS, smem, s>>>(n, rank, nout, a1, ld, (const __nv_bfloat16*)a2, (const __nv_bfloat16*)bias, 1.f / tau, decay);
+    else gla_decay_kernel<<<grid, GD_THREADS, smem, s>>>(n, rank, nout, a1, ld, (const float*)a2, (const float*)bias, 1.f / tau, decay);
+    return launch_check(cudaGetLastError(), "gla_decay");
 }
 
 int launch_ssd_prep(int dt, int n, int H, const float* dt_raw, int ld, const void* A_log, const void* dt_bias, float* step, float* decay, cudaStream_t s) {

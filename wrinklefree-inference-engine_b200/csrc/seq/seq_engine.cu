@@ -68,6 +68,14 @@ struct LayerState {
     // gated recurrences: the two gate biases (element-wise: z.b, x.b; matrix memory: i.b, f.b); state offset of the running maximum
     void *gb1 = nullptr, *gb2 = nullptr;
     size_t st_m = 0;
+    // one input product for the whole layer (wf_seq_config.one_norm): its rows (0: the mixer has a product of its own), this mixer's first
+    // column in it, and the branch gates' first column; biases of the branch gates and of layer norms; output norms of a pair
+    int in_np = 0, in_col = 0, rg_col = 0;
+    void *rg1_b = nullptr, *rg2_b = nullptr, *norm1_bias = nullptr, *norm2_bias = nullptr, *out_norm = nullptr, *pair_out_norm = nullptr;
+    // attention: learned numbers of the logarithmic distance penalty, head mixture — as loaded and as floats (made at finalize; sink_f above);
+    // gated linear attention: decay bias
+    void *r1_raw = nullptr, *r2_raw = nullptr, *talk_raw = nullptr, *a2_bias = nullptr;
+    float *r1_f = nullptr, *r2_f = nullptr, *talk_f = nullptr;
     // state slot offsets (floats)
     size_t st_canon1 = 0, st_canon2 = 0, st_conv = 0, st_S = 0;
 };
@@ -82,7 +90,7 @@ struct wf_seq_engine {
     std::vector<LayerState> layers;
     std::vector<TensorSlot> tensors;
     std::map<std::string, int> tensor_index;
-    void *embed = nullptr, *final_norm = nullptr, *head = nullptr;
+    void *embed = nullptr, *final_norm = nullptr, *head = nullptr, *pos_table = nullptr, *final_norm_b = nullptr;
     bool finalized = false;
     // cache + state
     PageTable pt;
@@ -116,6 +124,7 @@ struct wf_seq_engine {
     int attn_waves = 4;               // decode attention: resident waves of CTAs the key splits aim at (WF_SEQ_ATTN_WAVES)
     float* gqa_ws = nullptr;          // partial results of key-split grouped-query attention: gqa_ws_rows (token, head, split) rows
     int gqa_ws_rows = 0;
+    size_t gqa_ws_bytes = 0;
     float* attn_ws = nullptr;         // partial results of key-split attention
     int attn_ws_rows = 0;             // token-splits it holds
     int pair_path_max = 64;           // up to this many (token, expert) pairs the experts run as per-pair weight streams (WF_SEQ_PAIR_MAX)
@@ -170,6 +179,13 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
         return WF_ERR_INVALID;
     }
     if (c.block_form != WF_SEQ_BLOCK_SANDWICH && c.block_form != WF_SEQ_BLOCK_POST && c.block_form != WF_SEQ_BLOCK_PARALLEL) { set_error("wf_seq_create: block form %d", c.block_form); return WF_ERR_INVALID; }
+    const bool par = c.block_form == WF_SEQ_BLOCK_PARALLEL;
+    if (!par && (c.layer_norm || c.one_norm || c.branch_gates)) { set_error("wf_seq_create: layer norms with biases, one norm for both branches and branch gates belong to the parallel block form"); return WF_ERR_UNSUPPORTED; }
+    if (c.branch_gates && !c.one_norm) { set_error("wf_seq_create: branch gates read the one norm of the layer"); return WF_ERR_UNSUPPORTED; }
+    if (c.layer_norm && (!c.one_norm || c.norm_offset != 0.f)) { set_error("wf_seq_create: layer norms come one per layer, with plain weights"); return WF_ERR_UNSUPPORTED; }
+    if (c.pos_embed < 0 || c.pos_embed > 2 || (c.pos_embed == 2 && c.max_positions <= 0) || (c.pos_embed == 1 && c.block_form != WF_SEQ_BLOCK_POST) || c.logit_softcap < 0.f) {
+        set_error("wf_seq_create: position embedding %d (%d positions), logit cap %g", c.pos_embed, c.max_positions, c.logit_softcap); return WF_ERR_INVALID;
+    }
     if (c.page_size <= 0 || c.max_pages <= 0 || c.slots <= 0 || c.max_step_tokens <= 0) { set_error("wf_seq_create: page / slot / step sizes must be positive"); return WF_ERR_INVALID; }
     if (c.n_extra < 0) { set_error("wf_seq_create: %d extra mixers", c.n_extra); return WF_ERR_INVALID; }
     for (int i = 0; i < c.n_layers + c.n_extra; ++i) {
@@ -196,6 +212,8 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
             if (l.heads != 1 || l.dim != 1) { set_error("layer %d: the element-wise recurrence has heads = dim = 1 and vdim channels", i); return WF_ERR_INVALID; }
         } else if (l.type == WF_SEQ_MLSTM) {
             if (l.gate_cap < 0.f) { set_error("layer %d: gate cap %g", i, l.gate_cap); return WF_ERR_INVALID; }
+        } else if (l.type == WF_SEQ_GLA) {
+            if (l.decay_rank <= 0 || !(l.decay_tau > 0.f)) { set_error("layer %d: decay rank %d, tau %g", i, l.decay_rank, l.decay_tau); return WF_ERR_INVALID; }
         } else if (l.type == WF_SEQ_DELTA) {
             if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.conv < 1 || l.decay_rank < 0 || l.gate_rank < 0) { set_error("layer %d: delta sizes", i); return WF_ERR_INVALID; }
         } else if (l.type == WF_SEQ_SSD) {
@@ -203,7 +221,7 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
         } else if (l.type == WF_SEQ_GQA_ATTENTION) {
             if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.window < 1) { set_error("layer %d: attention sizes", i); return WF_ERR_INVALID; }
             if (l.v_is_k && (l.vdim != l.dim || l.v_norm || l.kv_from >= 0)) { set_error("layer %d: values that are the keys have the keys' size, no norm of their own and a cache of their own", i); return WF_ERR_INVALID; }
-            if (l.sink < 0 || l.sink > 1) { set_error("layer %d: grouped-query attention takes no sink or the extra one", i); return WF_ERR_INVALID; }
+            if (l.sink < 0 || l.sink > 2) { set_error("layer %d: sink kind %d", i, l.sink); return WF_ERR_INVALID; }
             if (l.qk_norm < 0 || l.qk_norm > 3 || l.rope_dims < 0 || (l.rope_dims & 1) || l.rope_dims > l.dim || l.chunk < 0 || l.rel_rows < 0 || l.softcap < 0.f ||
                 (l.rel_rows > 0 && (l.rel_rows < 2 || !(l.rel_far > (float)(l.rel_rows / 2)))) || l.head_gate < 0 || l.head_gate > 2 || l.proj_bias < 0 || l.proj_bias > 2) {
                 set_error("layer %d: attention options", i); return WF_ERR_INVALID;
@@ -216,6 +234,8 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
                 }
             }
         } else { set_error("layer %d: unknown mixer type %d", i, l.type); return WF_ERR_INVALID; }
+        if (c.one_norm && l.type != WF_SEQ_GQA_ATTENTION && l.type != WF_SEQ_GLA) { set_error("layer %d: mixer type %d does not take the layer's one input product", i, l.type); return WF_ERR_UNSUPPORTED; }
+        if (l.pair_norm && !l.pair) { set_error("layer %d: output norms of a pair without a second mixer", i); return WF_ERR_INVALID; }
         if (l.has_ff != WF_SEQ_FF_NONE && l.has_ff != WF_SEQ_FF_ROUTED && l.has_ff != WF_SEQ_FF_DENSE) { set_error("layer %d: feed-forward kind %d", i, l.has_ff); return WF_ERR_INVALID; }
         if (l.has_ff == WF_SEQ_FF_DENSE && l.ff <= 0) { set_error("layer %d: dense feed-forward size", i); return WF_ERR_INVALID; }
         if (l.ff_act == WF_SEQ_ACT_RELU2 && l.has_ff != WF_SEQ_FF_DENSE && l.has_ff != WF_SEQ_FF_NONE) { set_error("layer %d: the ungated activation belongs to a dense feed-forward", i); return WF_ERR_INVALID; }
@@ -263,6 +283,9 @@ int prepare_step(wf_seq_engine* e, int nseq, const int32_t* slots, const int32_t
     if (nwant < 0 || nwant > n) { set_error("wf_seq_step: %d wanted rows of %d tokens", nwant, n); return WF_ERR_INVALID; }
     for (int j = 0; j < nwant; ++j) if (want[j] < 0 || want[j] >= n) { set_error("wf_seq_step: wanted row %d out of range", want[j]); return WF_ERR_INVALID; }
     if (tokens) for (int i = 0; i < n; ++i) if (tokens[i] < 0 || tokens[i] >= c.vocab) { set_error("wf_seq_step: token id %d outside the vocabulary", tokens[i]); return WF_ERR_INVALID; }
+    if (c.pos_embed == 2)
+        for (int i = 0; i < nseq; ++i)
+            if (e->h_len[slots[i]] + counts[i] > c.max_positions) { set_error("wf_seq_step: sequence %d would reach position %d of %d", i, e->h_len[slots[i]] + counts[i] - 1, c.max_positions); return WF_ERR_INVALID; }
     // pages for the new tokens (all or nothing)
     for (int i = 0; i < nseq; ++i) {
         if (!e->pt.ensure(slots[i], e->h_len[slots[i]] + counts[i])) {
@@ -304,10 +327,25 @@ void commit_lengths(wf_seq_engine* e, int nseq, const int32_t* slots, const int3
     for (int i = 0; i < nseq; ++i) e->h_len[slots[i]] += counts[i];
 }
 
+// rows that a mixer adds to a layer's one input product
+int one_norm_rows(const wf_seq_layer& l) {
+    const int nk = l.heads * l.dim, nv = l.heads * l.vdim;
+    if (l.type == WF_SEQ_GLA) return 2 * nk + 2 * nv + l.decay_rank;
+    return nk + (l.kv_from < 0 ? l.kv_heads * (l.dim + (l.v_is_k ? 0 : l.vdim)) : 0) + (l.head_gate == 2 ? nv : l.head_gate ? l.heads : 0);
+}
+
 GemmArgs lin(const void* A, int a_f32, int lda, const void* B, int ldb, void* C, int c_f32, int ldc, int M, int N, int K) {
     GemmArgs g;
     g.A = A; g.a_f32 = a_f32; g.lda = lda; g.B = B; g.ldb = ldb; g.C = C; g.c_f32 = c_f32; g.ldc = ldc; g.M = M; g.N = N; g.K = K;
     return g;
+}
+
+// where a mixer finds its input projection: columns of the layer's one input product, or a product of its own
+int in_proj(wf_seq_engine* e, const LayerState& L, const Batch& b, const float** pj, int* ld) {
+    if (L.in_np) { *pj = e->proj + L.in_col; *ld = L.in_np; return WF_OK; }
+    *pj = e->proj; *ld = L.np;
+    const int W = e->cfg.width;
+    return launch_gemm(e->dt, lin(e->h_t, 0, W, L.wp, W, e->proj, 1, L.np, b.n, L.np, W), e->stream);
 }
 
 // h (post-convolution input, storage type [n, W]) -> y float [n, W]
@@ -447,21 +485,35 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     D.q_norm_w = L.q_norm_w; D.k_norm_w = L.k_norm_w;
     D.chunk = c.chunk; D.sink = c.sink; D.gate_elem = c.head_gate == 2; D.softcap = c.softcap;
     D.rel = L.rel_dist; D.rel_n = L.rel_n; D.v_is_k = c.v_is_k;
+    D.dist_r1 = L.r1_f; D.dist_r2 = L.r2_f; D.sink_h = L.sink_f; D.talk = L.talk_f;
     const LayerState& src = c.kv_from >= 0 ? e->layers[c.kv_from] : L;        // whose cache rows this layer reads
     PagedCache pc{e->pool, e->page_stride, src.cache_off, e->cfg.page_size, e->d_block_table, e->pt.max_blocks};
-    if ((rc = launch_gemm(e->dt, lin(e->h_t, 0, W, L.wp, W, e->proj, 1, L.np, n, L.np, W), s))) return rc;     // [q | k | v | g]
+    const float* pj;
+    int ld;
+    if ((rc = in_proj(e, L, b, &pj, &ld))) return rc;     // [q | k | v | g]
     mark(e, "attn.proj_gemm");
-    if ((rc = launch_gqa_prep(e->dt, b, D, e->proj, L.np, L.k_off, L.v_off, L.g_off, L.qb, L.kb, L.vb, e->cfg.eps, pc, e->qn, c.head_gate ? e->gate : nullptr, s))) return rc;
+    if ((rc = launch_gqa_prep(e->dt, b, D, pj, ld, L.k_off, L.v_off, L.g_off, L.qb, L.kb, L.vb, e->cfg.eps, pc, e->qn, c.head_gate ? e->gate : nullptr, s))) return rc;
     mark(e, "attn.prep+kv_write");
     const float* gate = c.head_gate ? e->gate : nullptr;
-    if (e->dt == WF_BF16 && e->attn_mma >= 1 && gqa_attn_mma_usable(D, pc) && gqa_attn_mma_takes(D)) {
-        // decoding (one token per sequence): few CTAs with long key ranges, so the keys are cut until there are about four resident
-        // waves of CTAs (two are resident per SM): the machine is covered and the last wave's tail stays short.
-        // The cut depends on the batch size and the pool only, never on the lengths: a captured step stays valid.
+    // decoding (one token per sequence) cuts the key range over blocks; the cut depends on the batch size and the pool only, never on the
+    // lengths: a captured step stays valid
+    long long span = std::min<long long>(c.window, (long long)e->cfg.max_pages * e->cfg.page_size);
+    if (c.chunk > 0 && c.chunk < span) span = c.chunk;
+    if (e->dt == WF_BF16 && e->attn_mma >= 1 && D.talk && !gate && talk_attn_mma_usable(D, pc)) {
         int splits = 1;
         if (n == b.nseq) {
-            long long span = std::min<long long>(c.window, (long long)e->cfg.max_pages * e->cfg.page_size);
-            if (c.chunk > 0 && c.chunk < span) span = c.chunk;
+            splits = (2 * sm_count() + n - 1) / n;           // one block per token and split runs every head; one is resident per SM
+            if (splits > span / 128) splits = (int)(span / 128);
+            while (splits > 1 && talk_attn_workspace(D, n, splits) > e->gqa_ws_bytes) --splits;
+            if (splits > 64) splits = 64;
+            if (splits < 1) splits = 1;
+        }
+        if ((rc = launch_talk_attn_mma(b, D, e->qn, pc, e->og, e->gqa_ws, splits, s))) return rc;
+    } else if (e->dt == WF_BF16 && e->attn_mma >= 1 && gqa_attn_mma_usable(D, pc) && gqa_attn_mma_takes(D)) {
+        // decoding (one token per sequence): few CTAs with long key ranges, so the keys are cut until there are about four resident
+        // waves of CTAs (two are resident per SM): the machine is covered and the last wave's tail stays short.
+        int splits = 1;
+        if (n == b.nseq) {
             const int ctas = n * c.kv_heads, resident = 2 * sm_count();
             splits = (e->attn_waves * resident + ctas - 1) / ctas;
             if (splits > span / 256) splits = (int)(span / 256);
@@ -471,7 +523,7 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
         }
         if ((rc = launch_gqa_attn_mma(b, D, e->qn, gate, pc, e->og, e->gqa_ws, splits, s))) return rc;
     } else if ((rc = launch_gqa_attn(e->dt, b, D, e->qn, gate, pc, e->og, s))) return rc;
-    mark(e, D.softcap > 0.f || D.rel ? "attn.attention(cap+bias)" : "attn.attention");
+    mark(e, D.talk ? "attn.attention(mixed heads)" : D.softcap > 0.f || D.rel ? "attn.attention(cap+bias)" : "attn.attention");
     rc = launch_gemm(e->dt, lin(e->og, 0, nv, L.wo, nv, out, 1, W, n, W, nv), s);
     // the single-gain norm of the post form takes the bias itself, except for paired mixers (their outputs are combined first)
     if (!rc && L.ob && !(e->cfg.block_form == WF_SEQ_BLOCK_POST && !e->cfg.norm_weights && !L.c.pair && out == e->y)) rc = launch_add_bias(e->dt, out, W, L.ob, n, W, s);
@@ -516,8 +568,33 @@ int run_mlstm(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     return rc;
 }
 
+// gated linear attention: [q | k | v | g | a1] projection -> per-channel decays -> the plain recurrence with one decay per key row ->
+// per-head norm, silu gate -> output
+int run_gla(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
+    const wf_seq_layer& c = L.c;
+    const int W = e->cfg.width, n = b.n, H = c.heads, nk = H * c.dim, nv = H * c.vdim;
+    cudaStream_t s = e->stream;
+    int rc;
+    const float* pj;
+    int ld;
+    if ((rc = in_proj(e, L, b, &pj, &ld))) return rc;
+    mark(e, "gla.proj_gemm");
+    if ((rc = launch_gla_decay(e->dt, n, c.decay_rank, nk, pj + L.a_col, ld, L.a2, L.a2_bias, c.decay_tau, e->decay, s))) return rc;
+    mark(e, "gla.decay");
+    DeltaDims D{H, H, c.dim, c.vdim};
+    D.no_delta = 1; D.vec_decay = 1; D.q_off = 0; D.k_off = nk; D.v_off = 2 * nk; D.o_scale = 1.f / sqrtf((float)c.dim);
+    if ((rc = launch_delta_rule(b, D, pj, ld, nullptr, e->decay, e->state + L.st_S, e->slot_stride, e->od, s, &e->scan))) return rc;
+    mark(e, "gla.recurrence");
+    if ((rc = launch_delta_post(e->dt, D, n, e->od, L.onorm, e->cfg.eps, pj + L.g_col, ld, e->og, s, 0))) return rc;
+    mark(e, "gla.post");
+    rc = launch_gemm(e->dt, lin(e->og, 0, nv, L.wo, nv, out, 1, W, n, W, nv), s);
+    mark(e, "gla.out_gemm");
+    return rc;
+}
+
 int run_one_mixer(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     switch (L.c.type) {
+        case WF_SEQ_GLA: return run_gla(e, L, b, out);
         case WF_SEQ_MINGRU: return run_mingru(e, L, b, out);
         case WF_SEQ_MLSTM: return run_mlstm(e, L, b, out);
         case WF_SEQ_GQA_ATTENTION: return run_gqa(e, L, b, out);
@@ -531,10 +608,20 @@ int run_one_mixer(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
 // outputs are combined in float, here or (combine = false) by the norm kernel that follows.
 int run_mixer(wf_seq_engine* e, LayerState& L, const Batch& b, bool combine = true) {
     int rc;
+    if (L.in_np) {               // the layer's one input product: both mixers' projections and the branch gates' logits
+        const int W = e->cfg.width;
+        if ((rc = launch_gemm(e->dt, lin(e->h_t, 0, W, L.wp, W, e->proj, 1, L.in_np, b.n, L.in_np, W), e->stream))) return rc;
+        mark(e, "layer.proj_gemm");
+    }
     if ((rc = run_one_mixer(e, L, b, e->y))) return rc;
     if (!L.c.pair) return WF_OK;
     if ((rc = run_one_mixer(e, e->layers[L.pair_state], b, e->y2))) return rc;
     if (!combine) return WF_OK;                  // the caller's norm kernel forms mix_scale * y + pair_scale * y2 on its way in
+    if (L.c.pair_norm) {
+        const int W = e->cfg.width;
+        if ((rc = launch_group_rmsnorm(e->dt, e->y, W, L.out_norm, 1, e->cfg.eps, b.n, W, nullptr, e->y, W, nullptr, 0, nullptr, e->stream))) return rc;
+        if ((rc = launch_group_rmsnorm(e->dt, e->y2, W, L.pair_out_norm, 1, e->cfg.eps, b.n, W, nullptr, e->y2, W, nullptr, 0, nullptr, e->stream))) return rc;
+    }
     rc = launch_axpby(e->y, L.c.mix_scale, e->y2, L.c.pair_scale, (size_t)b.n * e->cfg.width, e->stream);
     mark(e, "pair.combine");
     return rc;
@@ -651,16 +738,24 @@ int run_input(wf_seq_engine* e, const Batch& b, const void* norm_w, const void* 
 
 // WF_SEQ_BLOCK_POST: every sublayer reads the stream itself (h_t is its storage-type copy, refreshed by the kernel that updates the stream)
 // and its output is normalised with one gain, scaled and added.
+// the scaled embedding rows, with the learned position vectors where the model has them, into the stream (and its storage-type copy)
+int run_embed(wf_seq_engine* e, const StepView& v, void* x_t = nullptr) {
+    const float escale = e->cfg.embed_scale != 0.f ? e->cfg.embed_scale : 1.f;
+    const int rc = launch_embed_f32(e->dt, e->embed, v.tokens, v.b.n, e->cfg.width, e->x, e->stream, escale, x_t, e->pos_table, v.b.tok_pos);
+    mark(e, "embed");
+    return rc;
+}
+
 int run_layers_post(wf_seq_engine* e, const StepView& v) {
     const int W = e->cfg.width, n = v.b.n;
     const float mult = e->cfg.residual_mult, eps = e->cfg.eps;
     cudaStream_t s = e->stream;
     int rc;
-    const float escale = e->cfg.embed_scale != 0.f ? e->cfg.embed_scale : 1.f;
     const bool vec = e->cfg.norm_weights != 0;            // weight vectors (one launch of the grouped norm with one group) or single gains
-    if (e->cfg.pos_embed) { if ((rc = launch_embed_pos(e->dt, e->embed, v.tokens, v.b.tok_pos, n, W, e->cfg.pos_base, e->x, e->h_t, s))) return rc; }
-    else if ((rc = launch_embed_f32(e->dt, e->embed, v.tokens, n, W, e->x, s, escale, e->h_t))) return rc;
-    mark(e, "embed");
+    if (e->cfg.pos_embed == 1) {
+        if ((rc = launch_embed_pos(e->dt, e->embed, v.tokens, v.b.tok_pos, n, W, e->cfg.pos_base, e->x, e->h_t, s))) return rc;
+        mark(e, "embed");
+    } else if ((rc = run_embed(e, v, e->h_t))) return rc;
     for (int li = 0; li < e->cfg.n_layers; ++li) {
         LayerState& L = e->layers[li];
         if ((rc = run_mixer(e, L, v.b, !vec))) return rc;
@@ -690,9 +785,7 @@ int run_layers_parallel(wf_seq_engine* e, const StepView& v) {
     const float eps = e->cfg.eps, off = e->cfg.norm_offset;
     cudaStream_t s = e->stream;
     int rc;
-    const float escale = e->cfg.embed_scale != 0.f ? e->cfg.embed_scale : 1.f;
-    if ((rc = launch_embed_f32(e->dt, e->embed, v.tokens, n, W, e->x, s, escale))) return rc;
-    mark(e, "embed");
+    if ((rc = run_embed(e, v))) return rc;
     {
         LayerState& L0 = e->layers[0];
         if ((rc = launch_add_dual_norm(e->dt, e->x, nullptr, 0.f, nullptr, 0.f, nullptr, L0.norm1, L0.c.has_ff ? L0.norm2 : nullptr, off, eps, n, W, e->h_t, e->h_t2, s))) return rc;
@@ -713,14 +806,42 @@ int run_layers_parallel(wf_seq_engine* e, const StepView& v) {
     return WF_OK;
 }
 
+// The same form with ONE norm per layer whose output both branches read, and optionally a sigmoid gate per branch and element: one kernel
+// per layer boundary norms and combines the pair's outputs, gates both branches, adds them to the stream and forms the next layer's input.
+int run_layers_one_norm(wf_seq_engine* e, const StepView& v) {
+    const int W = e->cfg.width, n = v.b.n, NL = e->cfg.n_layers;
+    const float eps = e->cfg.eps, off = e->cfg.norm_offset;
+    cudaStream_t s = e->stream;
+    int rc;
+    if ((rc = run_embed(e, v))) return rc;
+    if ((rc = launch_branch_add_norm(e->dt, e->x, BranchSum(), e->layers[0].norm1, e->layers[0].norm1_bias, off, eps, n, W, e->h_t, s))) return rc;
+    mark(e, "residual+norm");
+    for (int li = 0; li < NL; ++li) {
+        LayerState& L = e->layers[li];
+        if ((rc = run_mixer(e, L, v.b, false))) return rc;
+        if (L.c.has_ff && (rc = run_unit(e, L, v.b, e->uy))) return rc;
+        BranchSum bs;
+        bs.y1 = e->y; bs.y3 = L.c.has_ff ? e->uy : nullptr;
+        if (L.c.pair) { bs.y2 = e->y2; bs.a1 = L.c.mix_scale; bs.a2 = L.c.pair_scale; bs.pw1 = L.out_norm; bs.pw2 = L.pair_out_norm; }
+        if (e->cfg.branch_gates) { bs.gate = e->proj + L.rg_col; bs.ldg = L.in_np; bs.gb1 = L.rg1_b; bs.gb2 = L.rg2_b; }
+        const LayerState* N = li + 1 < NL ? &e->layers[li + 1] : nullptr;
+        if ((rc = launch_branch_add_norm(e->dt, e->x, bs, N ? N->norm1 : nullptr, N ? N->norm1_bias : nullptr, off, eps, n, W, e->h_t, s))) return rc;
+        mark(e, "residual+norm");
+        if (e->layer_tap) {
+            if (cuda_check(cudaMemcpyAsync(e->layer_tap + (size_t)li * n * W, e->x, (size_t)n * W * 4, cudaMemcpyDeviceToHost, s), "layer tap")) return WF_ERR_CUDA;
+        }
+    }
+    return WF_OK;
+}
+
 int run_layers(wf_seq_engine* e, const StepView& v) {
+    if (e->cfg.one_norm) return run_layers_one_norm(e, v);
     if (e->cfg.block_form == WF_SEQ_BLOCK_POST) return run_layers_post(e, v);
     if (e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL) return run_layers_parallel(e, v);
     const int W = e->cfg.width, n = v.b.n;
     cudaStream_t s = e->stream;
     int rc;
-    if ((rc = launch_embed_f32(e->dt, e->embed, v.tokens, n, W, e->x, s))) return rc;
-    mark(e, "embed");
+    if ((rc = run_embed(e, v))) return rc;
     for (int li = 0; li < e->cfg.n_layers; ++li) {
         LayerState& L = e->layers[li];
         if ((rc = run_input(e, v.b, L.norm1, L.canon1, L.st_canon1))) return rc;
@@ -757,12 +878,14 @@ int run_head(wf_seq_engine* e, const StepView& v, int nwant) {
     const int W = e->cfg.width;
     int rc;
     if ((rc = ensure_logits(e, nwant))) return rc;
-    if (e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL) rc = launch_group_rmsnorm(e->dt, e->x, W, e->final_norm, 1, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream, nullptr, 1.f, 0.f, e->cfg.norm_offset);
+    if (e->cfg.layer_norm) rc = launch_layer_norm(e->dt, e->x, W, e->final_norm, e->final_norm_b, e->cfg.eps, nwant, W, nullptr, W, e->xn, W, v.want, e->stream);
+    else if (e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL) rc = launch_group_rmsnorm(e->dt, e->x, W, e->final_norm, 1, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream, nullptr, 1.f, 0.f, e->cfg.norm_offset);
     else if (e->cfg.block_form == WF_SEQ_BLOCK_POST && e->cfg.norm_weights) rc = launch_group_rmsnorm(e->dt, e->x, W, e->final_norm, 1, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream);
     else if (e->cfg.block_form == WF_SEQ_BLOCK_POST) rc = launch_scalar_rmsnorm(e->dt, e->x, W, nullptr, e->final_norm, 1.f, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream);
     else rc = launch_group_rmsnorm(e->dt, e->x, W, e->final_norm, e->cfg.norm_groups, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream);
     if (rc) return rc;
     rc = launch_gemm(e->dt, lin(e->xn, 0, W, e->head, W, e->logits, 1, e->cfg.vocab, nwant, e->cfg.vocab, W), e->stream);
+    if (!rc && e->cfg.logit_softcap > 0.f) rc = launch_softcap(e->logits, (size_t)nwant * e->cfg.vocab, e->cfg.logit_softcap, e->stream);
     mark(e, "final_norm+head_gemm");
     return rc;
 }
@@ -835,6 +958,8 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
     TRY(dalloc_t(e, &e->final_norm, norm_elems));
     add_tensor(e, "embed", e->embed, (size_t)c.vocab * W);
     add_tensor(e, "final.norm", e->final_norm, norm_elems);
+    if (c.layer_norm) { TRY(dalloc_t(e, &e->final_norm_b, W)); add_tensor(e, "final.norm.b", e->final_norm_b, W); }
+    if (c.pos_embed == 2) { TRY(dalloc_t(e, &e->pos_table, (size_t)c.max_positions * W)); add_tensor(e, "pos", e->pos_table, (size_t)c.max_positions * W); }
     if (c.tied_head) e->head = e->embed;
     else { TRY(dalloc_t(e, &e->head, (size_t)c.vocab * W)); add_tensor(e, "head", e->head, (size_t)c.vocab * W); }
     // maxima over layers for the shared workspaces
@@ -843,6 +968,7 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
     size_t st = 0;
     e->layers.resize(c.n_layers + c.n_extra);
     size_t max_gate = 1, max_decay = 1, max_gfull = 0, max_afull = 0, max_scan = 0, max_qfull = 0, max_qrank = 0;
+    size_t max_talk_ws = 0;          // mixed heads: one unsplit partial result for every sequence, and room for one per SM
     bool any_mlstm = false;
     bool own = true;                 // false while a tied layer is laid out: it allocates and names nothing, its weights are its source's
     auto walloc = [&](void** ptr, size_t count) -> int { return own ? dalloc_t(e, ptr, count) : WF_OK; };
@@ -864,7 +990,7 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
             if (ownv) { L.v_off = (int)off; off += nvk; }
             if (l.head_gate) { L.g_off = (int)off; off += ng; }
             L.np = (int)off;
-            TRYL(walloc(&L.wp, (size_t)L.np * W));
+            if (!L.in_np) TRYL(walloc(&L.wp, (size_t)L.np * W));
             name(mp + "q", L.wp, nq * W);
             if (ownkv) {
                 name(mp + "k", at(e, L.wp, (size_t)L.k_off * W), nk * W);
@@ -884,6 +1010,19 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
                 TRYL(walloc(&L.q_norm_w, wq)); name(mp + "q.norm", L.q_norm_w, wq);
                 TRYL(walloc(&L.k_norm_w, wk)); name(mp + "k.norm", L.k_norm_w, wk);      // a layer that reads another's cache still names it: unused
             }
+            if (l.dist_log) {
+                TRYL(walloc(&L.r1_raw, l.heads)); name(mp + "r1", L.r1_raw, l.heads);
+                TRYL(walloc(&L.r2_raw, l.heads)); name(mp + "r2", L.r2_raw, l.heads);
+                if (own) { TRYL(dalloc_n(e, &L.r1_f, l.heads)); TRYL(dalloc_n(e, &L.r2_f, l.heads)); }
+            }
+            if (l.sink == 2) {
+                TRYL(walloc(&L.sink_raw, l.heads)); name(mp + "sink", L.sink_raw, l.heads);
+                if (own) TRYL(dalloc_n(e, &L.sink_f, l.heads));
+            }
+            if (l.talk) {
+                TRYL(walloc(&L.talk_raw, (size_t)l.heads * l.heads)); name(mp + "talk", L.talk_raw, (size_t)l.heads * l.heads);
+                if (own) TRYL(dalloc_n(e, &L.talk_f, (size_t)l.heads * l.heads));
+            }
             if (l.rel_rows > 0) {
                 TRYL(walloc(&L.rel, (size_t)l.rel_rows * l.heads)); name(mp + "rel", L.rel, (size_t)l.rel_rows * l.heads);
                 // beyond rel_far every distance falls into the last row: rel_far + 1 rows by distance are all there is
@@ -895,6 +1034,10 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
                 cache_elems = (cache_elems + 7) / 8 * 8;
                 L.cache_off = cache_elems;
                 cache_elems += (long long)c.page_size * (nk + (ownv ? nvk : 0));
+            }
+            if (l.talk) {
+                GqaDims T{l.heads, l.kv_heads, l.dim, l.vdim, 0.f, 0.f, 1, 0, 0};
+                max_talk_ws = std::max(max_talk_ws, talk_attn_workspace(T, std::max(c.slots, 2 * sm_count()), 1));
             }
             max_hd = std::max(max_hd, nq); max_gqa_dv = std::max(max_gqa_dv, (size_t)l.vdim);
             max_gate = std::max(max_gate, ng);
@@ -955,6 +1098,24 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
             max_scan = std::max(max_scan, (size_t)l.heads * l.dim * (l.vdim + 1));
             max_hv = std::max(max_hv, (size_t)l.heads * (l.vdim + 1));
             any_mlstm = true;
+        } else if (l.type == WF_SEQ_GLA) {
+            // [q | k | v | g | first factor of the decay]; state: one matrix per head
+            const size_t nk = (size_t)l.heads * l.dim;
+            L.n_decay = (int)nk;
+            L.g_col = (int)(2 * nk + nv); L.a_col = (int)(2 * nk + 2 * nv);
+            L.np = L.a_col + l.decay_rank;
+            if (!L.in_np) TRYL(walloc(&L.wp, (size_t)L.np * W));
+            name(mp + "q", L.wp, nk * W);
+            name(mp + "k", at(e, L.wp, nk * W), nk * W);
+            name(mp + "v", at(e, L.wp, 2 * nk * W), nv * W);
+            name(mp + "g", at(e, L.wp, (size_t)L.g_col * W), nv * W);
+            name(mp + "a1", at(e, L.wp, (size_t)L.a_col * W), (size_t)l.decay_rank * W);
+            TRYL(walloc(&L.a2, nk * l.decay_rank)); name(mp + "a2", L.a2, nk * l.decay_rank);
+            TRYL(walloc(&L.a2_bias, nk)); name(mp + "a2.b", L.a2_bias, nk);
+            TRYL(walloc(&L.onorm, l.vdim)); name(mp + "norm", L.onorm, l.vdim);
+            L.st_S = st; st += nk * l.vdim;
+            max_decay = std::max(max_decay, nk);
+            max_scan = std::max(max_scan, nk * l.vdim);
         } else if (l.type == WF_SEQ_SSD) {
             // [z | x | B | C | dt]: x, B and C are the convolved channels
             const size_t GN = (size_t)l.kv_heads * l.dim;
@@ -1020,7 +1181,8 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
         if (own) L.norm1 = L.norm2 = L.norm1b = L.norm2b = L.canon1 = L.canon2 = nullptr;
         if (post) {
             TRY(walloc(&L.norm1, lnorm)); name(p + "norm1", L.norm1, lnorm);
-            if (l.has_ff) { TRY(walloc(&L.norm2, lnorm)); name(p + "norm2", L.norm2, lnorm); }
+            if (c.layer_norm) { TRY(walloc(&L.norm1_bias, W)); name(p + "norm1.b", L.norm1_bias, W); }
+            if (l.has_ff && !c.one_norm) { TRY(walloc(&L.norm2, lnorm)); name(p + "norm2", L.norm2, lnorm); }
         } else {
             void** norms[4] = {&L.norm1, &L.norm1b, &L.norm2, &L.norm2b};
             const char* norm_names[4] = {"norm1", "norm1b", "norm2", "norm2b"};
@@ -1032,6 +1194,22 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
                 L.st_canon2 = st; st += (size_t)(taps - 1) * W;
             }
         }
+        if (c.one_norm && own) {
+            // one input product: [mixer | second mixer | branch gate | feed-forward's gate]
+            const int left = one_norm_rows(l), right = l.pair ? one_norm_rows(layers[l.pair]) : 0;
+            L.rg_col = left + right;
+            L.in_np = L.rg_col + (c.branch_gates ? (l.has_ff ? 2 : 1) * W : 0);
+            TRY(walloc(&L.wp, (size_t)L.in_np * W));
+            if (l.pair) { LayerState& R = e->layers[l.pair]; R.in_np = L.in_np; R.in_col = left; R.wp = at(e, L.wp, (size_t)left * W); }
+            if (c.branch_gates) {
+                name(p + "rg1", at(e, L.wp, (size_t)L.rg_col * W), (size_t)W * W);
+                TRY(walloc(&L.rg1_b, W)); name(p + "rg1.b", L.rg1_b, W);
+                if (l.has_ff) {
+                    name(p + "rg2", at(e, L.wp, ((size_t)L.rg_col + W) * W), (size_t)W * W);
+                    TRY(walloc(&L.rg2_b, W)); name(p + "rg2.b", L.rg2_b, W);
+                }
+            }
+        }
         TRY(setup_mixer(L, l.pair ? p + "mix.left." : p + "mix."));
         if (l.pair) {
             LayerState& R = e->layers[l.pair];
@@ -1039,7 +1217,12 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
             R.c = layers[l.pair];
             L.pair_state = l.pair;
             TRY(setup_mixer(R, p + "mix.right."));
+            if (l.pair_norm) {
+                TRY(walloc(&L.out_norm, W)); name(p + "mix.left.out", L.out_norm, W);
+                TRY(walloc(&L.pair_out_norm, W)); name(p + "mix.right.out", L.pair_out_norm, W);
+            }
         }
+        max_np = std::max(max_np, (size_t)L.in_np);
         if (l.has_ff == WF_SEQ_FF_DENSE) {
             L.uff = l.ff; L.ulimit = l.ff_limit;
             const bool gated = l.ff_act != WF_SEQ_ACT_RELU2;
@@ -1108,11 +1291,15 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
     if (max_scan && T >= 2 * SCAN_CHUNK) {
         e->scan.chunks = scan_chunks_needed(T, c.slots);
         TRY(dalloc_n(e, &e->scan.local, (size_t)e->scan.chunks * max_scan)); TRY(dalloc_n(e, &e->scan.start, (size_t)e->scan.chunks * max_scan));
-        TRY(dalloc_n(e, &e->scan.prod, (size_t)e->scan.chunks * max_H));
+        TRY(dalloc_n(e, &e->scan.prod, (size_t)e->scan.chunks * std::max(max_H, max_decay)));
     }
     if (max_gfull) TRY(dalloc_n(e, &e->gfull, (size_t)T * max_gfull));
     if (max_afull) TRY(dalloc_n(e, &e->afull, (size_t)T * max_afull));
-    if (e->dt == WF_BF16 && max_gqa_dv) { e->gqa_ws_rows = 32768; TRY(dalloc_bytes(e, (void**)&e->gqa_ws, gqa_attn_mma_workspace(e->gqa_ws_rows, 1, (int)max_gqa_dv))); }
+    if (e->dt == WF_BF16 && max_gqa_dv) {
+        e->gqa_ws_rows = 32768;
+        e->gqa_ws_bytes = std::max(gqa_attn_mma_workspace(e->gqa_ws_rows, 1, (int)max_gqa_dv), max_talk_ws);
+        TRY(dalloc_bytes(e, (void**)&e->gqa_ws, e->gqa_ws_bytes));
+    }
     if (max_uff) { TRY(dalloc_n(e, &e->ugu, (size_t)T * 2 * max_uff)); TRY(dalloc_t(e, &e->uhmid, (size_t)T * max_uff)); TRY(dalloc_n(e, &e->uy, (size_t)T * W)); }
     TRY(dalloc_n(e, &e->qkvc, (size_t)T * max_C)); TRY(dalloc_n(e, &e->beta, (size_t)T * max_H)); TRY(dalloc_n(e, &e->decay, (size_t)T * std::max(max_H, max_decay)));
     TRY(dalloc_n(e, &e->od, (size_t)T * max_hv));
@@ -1163,6 +1350,21 @@ extern "C" int wf_seq_set_tensor(wf_seq_engine* e, const char* name, const void*
     t.loaded = true;
     e->finalized = false;
     return WF_OK;
+}
+
+// dst float [count] = src (storage type), both on the device; nothing to do where the model has no such tensor
+static int to_floats(wf_seq_engine* e, const void* src, float* dst, size_t count) {
+    if (!src || !dst) return WF_OK;
+    std::vector<unsigned char> raw(count * e->esz);
+    if (cuda_check(cudaMemcpyAsync(raw.data(), src, raw.size(), cudaMemcpyDeviceToHost, e->stream), "tensor D2H")) return WF_ERR_CUDA;
+    if (cuda_check(cudaStreamSynchronize(e->stream), "sync")) return WF_ERR_CUDA;
+    std::vector<float> f(count);
+    for (size_t k = 0; k < count; ++k) {
+        if (e->dt == WF_F32) f[k] = ((const float*)raw.data())[k];
+        else { const uint32_t bits = (uint32_t)((const uint16_t*)raw.data())[k] << 16; memcpy(&f[k], &bits, 4); }
+    }
+    if (cuda_check(cudaMemcpyAsync(dst, f.data(), count * 4, cudaMemcpyHostToDevice, e->stream), "tensor H2D")) return WF_ERR_CUDA;
+    return cuda_check(cudaStreamSynchronize(e->stream), "sync");
 }
 
 extern "C" int wf_seq_finalize(wf_seq_engine* e) {
@@ -1223,18 +1425,16 @@ extern "C" int wf_seq_finalize(wf_seq_engine* e) {
             if (cuda_check(cudaMemcpyAsync(L.freq, f.data(), f.size() * sizeof(double), cudaMemcpyHostToDevice, e->stream), "rotation table H2D")) return WF_ERR_CUDA;
             if (cuda_check(cudaStreamSynchronize(e->stream), "sync")) return WF_ERR_CUDA;
         }
-        if (L.sink_f) {
-            std::vector<unsigned char> raw((size_t)l.heads * e->esz);
-            if (cuda_check(cudaMemcpyAsync(raw.data(), L.sink_raw, raw.size(), cudaMemcpyDeviceToHost, e->stream), "sinks D2H")) return WF_ERR_CUDA;
-            if (cuda_check(cudaStreamSynchronize(e->stream), "sync")) return WF_ERR_CUDA;
-            std::vector<float> sf(l.heads);
-            for (int h = 0; h < l.heads; ++h) {
-                if (e->dt == WF_F32) sf[h] = ((const float*)raw.data())[h];
-                else { const uint32_t bits = (uint32_t)((const uint16_t*)raw.data())[h] << 16; memcpy(&sf[h], &bits, 4); }
-            }
-            if (cuda_check(cudaMemcpyAsync(L.sink_f, sf.data(), sf.size() * 4, cudaMemcpyHostToDevice, e->stream), "sinks H2D")) return WF_ERR_CUDA;
-            if (cuda_check(cudaStreamSynchronize(e->stream), "sync")) return WF_ERR_CUDA;
-        }
+        if (int rc = to_floats(e, L.sink_raw, L.sink_f, l.heads)) return rc;
+    }
+    // grouped-query attention: learned penalty numbers, sinks and head mixture as floats
+    for (LayerState& L : e->layers) {
+        if (L.c.type != WF_SEQ_GQA_ATTENTION || L.c.tied) continue;
+        const size_t H = L.c.heads;
+        if (int rc = to_floats(e, L.r1_raw, L.r1_f, H)) return rc;
+        if (int rc = to_floats(e, L.r2_raw, L.r2_f, H)) return rc;
+        if (int rc = to_floats(e, L.sink_raw, L.sink_f, H)) return rc;
+        if (int rc = to_floats(e, L.talk_raw, L.talk_f, H * H)) return rc;
     }
     // tied latent layers use their source's tables
     for (LayerState& L : e->layers)
@@ -1318,9 +1518,13 @@ extern "C" int wf_seq_run_part(wf_seq_engine* e, int layer, int part, int nseq, 
     float* result = e->y;
     const bool parallel = e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL;
     const bool post = e->cfg.block_form == WF_SEQ_BLOCK_POST || parallel;
-    if (part == 5 && !(parallel && L.c.has_ff)) { set_error("wf_seq_run_part: layer %d has no second norm", layer); return WF_ERR_INVALID; }
+    if (part == 5 && !(parallel && L.c.has_ff && !e->cfg.one_norm)) { set_error("wf_seq_run_part: layer %d has no second norm", layer); return WF_ERR_INVALID; }
     if (post && (part == 1 || part == 4)) { set_error("wf_seq_run_part: this model's sublayers have no input convolution"); return WF_ERR_INVALID; }
-    if ((part == 0 || part == 5) && parallel) {
+    if (part == 0 && e->cfg.layer_norm) {
+        if (cuda_check(cudaMemcpyAsync(e->x, in_host, bytes, cudaMemcpyHostToDevice, s), "in")) return WF_ERR_CUDA;
+        rc = launch_layer_norm(e->dt, e->x, W, L.norm1, L.norm1_bias, e->cfg.eps, n, W, e->hn, W, nullptr, 0, nullptr, s);
+        result = e->hn;
+    } else if ((part == 0 || part == 5) && parallel) {
         if (cuda_check(cudaMemcpyAsync(e->x, in_host, bytes, cudaMemcpyHostToDevice, s), "in")) return WF_ERR_CUDA;
         rc = launch_group_rmsnorm(e->dt, e->x, W, part == 0 ? L.norm1 : L.norm2, 1, e->cfg.eps, n, W, nullptr, e->hn, W, nullptr, 0, nullptr, s, nullptr, 1.f, 0.f, e->cfg.norm_offset);
         result = e->hn;

@@ -9,8 +9,9 @@
 namespace wf {
 namespace seq {
 
-// x[i, :] = scale * table[tokens[i], :] as float; x_t: optional T copy
-int launch_embed_f32(int dt, const void* table, const int32_t* tokens, int n, int W, float* x, cudaStream_t s, float scale = 1.f, void* x_t = nullptr);
+// x[i, :] = scale * table[tokens[i], :] [+ pos_table[tok_pos[i], :]] as float; x_t: optional T copy
+int launch_embed_f32(int dt, const void* table, const int32_t* tokens, int n, int W, float* x, cudaStream_t s, float scale = 1.f, void* x_t = nullptr,
+                     const void* pos_table = nullptr, const int32_t* tok_pos = nullptr);
 // y = a * y + b * y2 over count floats
 int launch_axpby(float* y, float a, const float* y2, float b, size_t count, cudaStream_t s);
 // y = [res +] w * x / sqrt(mean_g(x^2) + eps) per row and per group of W / groups consecutive elements.  x, y, res float [n, W] with row
@@ -24,6 +25,25 @@ int launch_group_rmsnorm(int dt, const float* x, int ldx, const void* w, int gro
 // h1 = r * (w_offset + w1), h2 = r * (w_offset + w2) as T [n, W] (each optional: null weights).  The row statistics are formed once.
 int launch_add_dual_norm(int dt, float* x, const float* y1, float a1, const float* y2, float a2, const float* y3, const void* w1, const void* w2,
                          float w_offset, float eps, int n, int W, void* h1, void* h2, cudaStream_t s);
+// layer norm of the rows of x (float [n, W], row stride ldx; rows: optional gather): y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b as
+// float (y, stride ldy) and / or T (y_t, stride ldt)
+int launch_layer_norm(int dt, const float* x, int ldx, const void* w, const void* b, float eps, int n, int W, float* y, int ldy, void* y_t, int ldt,
+                      const int32_t* rows, cudaStream_t s);
+// The stream update of a layer whose branches are gated, and the next layer's input norm, in one kernel:
+//   m  = a1 * y1' + a2 * y2'        yk' = yk, or pwk * yk / sqrt(mean(yk^2) + eps) where the pair's outputs are normed (pw1 / pw2: T [W])
+//   x += s(gate[:, 0..W) + gb1) * m + s(gate[:, W..2W) + gb2) * y3      (gate float [n, ldg], s the logistic function; null: no gates)
+//   h  = norm(x): layer norm w * (x - mean) / sqrt(var + eps) + b (b not null), or RMS norm (w_offset + w) * x / sqrt(mean(x^2) + eps)
+// y2, y3, w optional; x, y* float [n, W] dense; h T [n, W].
+struct BranchSum {
+    const float *y1 = nullptr, *y2 = nullptr, *y3 = nullptr;
+    float a1 = 1.f, a2 = 1.f;
+    const void *pw1 = nullptr, *pw2 = nullptr;
+    const float* gate = nullptr; int ldg = 0;
+    const void *gb1 = nullptr, *gb2 = nullptr;
+};
+int launch_branch_add_norm(int dt, float* x, const BranchSum& bs, const void* w, const void* b, float w_offset, float eps, int n, int W, void* h, cudaStream_t s);
+// z <- cap * tanh(z / cap) over count floats
+int launch_softcap(float* z, size_t count, float cap, cudaStream_t s);
 // x[i, :] = table[tokens[i], :] + sinusoidal position vector of tok_pos[i] (entry 2k sin, 2k + 1 cos of pos * base^(-2k / W)); x_t: optional T copy
 int launch_embed_pos(int dt, const void* table, const int32_t* tokens, const int32_t* tok_pos, int n, int W, float base, float* x, void* x_t, cudaStream_t s);
 // x_t T [n, W] = x float [n, W] rounded to the storage type (dense rows)
@@ -122,7 +142,7 @@ int launch_transpose_heads(int dt, const void* in, int H, int R, int C, void* ou
 // T [d]), 3 RMS norm over the whole projection with weights T [H * d] / [G * d].  rope_dims > 0: the first rope_dims entries of every query
 // and key head are rotated after the norm (pairs (2i, 2i + 1) when rope_interleaved, else (i, i + rope_dims / 2)).  chunk > 0: a query sees
 // only keys of its own chunk of that many positions.  softcap > 0: score <- softcap * tanh(score / softcap).  rel (float [rel_n, H], on the
-// device): bias by distance, rel[min(i - j, rel_n - 1), h], added after the cap.  sink: the softmax denominator carries an extra 1.
+// device): bias by distance, rel[min(i - j, rel_n - 1), h], added after the cap.  sink = 1: the softmax denominator carries an extra 1.
 // gate_elem: the gate has one entry per output element ([n, H * dv]) instead of one per head ([n, H]).
 struct GqaDims {
     int H, G, d, dv; float scale, dist_exp; int window, qk_norm, v_norm;
@@ -131,6 +151,9 @@ struct GqaDims {
     int chunk = 0, sink = 0, gate_elem = 0; float softcap = 0.f;
     const float* rel = nullptr; int rel_n = 0;
     int v_is_k = 0;               // the values are the cached keys (dv == d): a page holds keys only, nothing is projected or stored for values
+    // dist_r1 / dist_r2 (float [H], device): score -= r1[h] ln(1 + r2[h] (i - j)).  sink_h (float [H], device; sink = 2): the denominator carries
+    // exp(sink_h[h]).  talk (float [H, H], device): the heads' weights are mixed before the value sum, w_h <- sum_g talk[h, g] w_g.
+    const float *dist_r1 = nullptr, *dist_r2 = nullptr, *sink_h = nullptr, *talk = nullptr;
 };
 // elements one layer's keys and values take in a cache page: keys [G][page_size][d], then values [G][page_size][dv]
 long long gqa_cache_elems(const GqaDims& D, int page_size);
@@ -144,6 +167,12 @@ int launch_gqa_prep(int dt, const Batch& b, const GqaDims& D, const float* proj,
 // sum, times gate[n, H] (null: no gate).
 int launch_gqa_attn(int dt, const Batch& b, const GqaDims& D, const void* qn, const float* gate, const PagedCache& pc, void* out, cudaStream_t s);
 
+// Attention whose heads' weights are mixed (D.talk) has kernels of its own: a plain one behind launch_gqa_attn, and tensor-core forms
+// (bf16 storage; seq_attn_talk.cu).  When every sequence brings one token the key range can be cut over `splits` CTAs; that form needs a
+// workspace of talk_attn_workspace(D, n, splits) bytes also for splits = 1.
+bool talk_attn_mma_usable(const GqaDims& D, const PagedCache& pc);
+size_t talk_attn_workspace(const GqaDims& D, int n, int splits);
+int launch_talk_attn_mma(const Batch& b, const GqaDims& D, const void* qn, const PagedCache& pc, void* out, float* workspace, int splits, cudaStream_t s);
 // the same on tensor cores (bf16 storage only; seq_attn_mma.cu): group sizes up to 16, per-head sizes multiples of 8 up to 128, cache rows
 // 16-byte aligned.  When every sequence brings one token the key range can be cut over `splits` CTAs; that needs a workspace of
 // gqa_attn_mma_workspace(n * H, splits, dv) bytes.
@@ -159,18 +188,22 @@ int launch_gqa_attn_mma(const Batch& b, const GqaDims& D, const void* qn, const 
 // u = beta v (a plain decayed outer-product accumulation: the state-space recurrence) instead of u = beta (v - S^T k).
 // ones_col (no_delta form): the state has one more column whose value input is 1 for every token, so that column dv of the output is
 // n . q with n the decayed sum of the written keys; state [H][d][dv + 1] and o [n, H, dv + 1] then.
-struct DeltaDims { int H, Hk, d, dv; int vec_decay = 0, no_delta = 0, q_off = -1, k_off = -1, v_off = -1, ones_col = 0; };
+// o_scale multiplies the read-out.
+struct DeltaDims { int H, Hk, d, dv; int vec_decay = 0, no_delta = 0, q_off = -1, k_off = -1, v_off = -1, ones_col = 0; float o_scale = 1.f; };
 // in place on qkv float [n, C = 2 * Hk * d + H * dv] (ld): q and k heads -> unit vectors (x / sqrt(sum x^2 + 1e-6)), q also times d^-1/2.
 // beta[n, H] = sigmoid(b_raw), decay[n, H] = exp(-exp(A_log[h]) * softplus(a_raw + dt_bias[h]))   (a_raw, b_raw float with strides);
 // with D.vec_decay a_raw and dt_bias have H * d entries and decay is [n, H, d]
 int launch_delta_prep(int dt, const DeltaDims& D, int n, float* qkv, int ld, const float* a_raw, int lda, const float* b_raw, int ldb_,
                       const void* A_log, const void* dt_bias, float* beta, float* decay, cudaStream_t s);
 // per (sequence, head): for each token in order  S = decay S;  u = beta (v - S^T k);  S += k u^T;  o = S^T q.   S float [slot][H][d][dv]
-// scan (optional, no_delta form with one decay per head only): long portions are cut into chunks of SCAN_CHUNK tokens that run in parallel —
+// (beta null: 1).  scan (optional, no_delta form only): long portions are cut into chunks of SCAN_CHUNK tokens that run in parallel —
 // every chunk's own contribution from a zero state, a short pass that chains the chunks' start states (S_start[c + 1] = prod_c S_start[c]
 // + local_c, the recurrence being linear in the state), then every chunk again from its start state for the outputs.
 constexpr int SCAN_CHUNK = 128;
-struct ScanWorkspace { float* local = nullptr; float* start = nullptr; float* prod = nullptr; int chunks = 0; };   // chunks: entries of H * d * dv floats each
+struct ScanWorkspace { float* local = nullptr; float* start = nullptr; float* prod = nullptr; int chunks = 0; };   // chunks: entries of H * d * dv floats each; prod: H (vec_decay: H * d) floats per chunk
+// gated linear attention: decay[i, c] = sigmoid(z)^(1 / tau), z = a2[c, :] . a1[i, :] + bias[c], c < nout; a1 float [n, rank] (ld), a2 T [nout, rank];
+// products, logarithm and exponential in float
+int launch_gla_decay(int dt, int n, int rank, int nout, const float* a1, int ld, const void* a2, const void* bias, float tau, float* decay, cudaStream_t s);
 inline int scan_chunks_needed(int max_step_tokens, int slots) { return max_step_tokens / SCAN_CHUNK + slots + 1; }
 int launch_delta_rule(const Batch& b, const DeltaDims& D, const float* qkv, int ld, const float* beta, const float* decay, float* state,
                       size_t slot_stride, float* o, cudaStream_t s, const ScanWorkspace* scan = nullptr);

@@ -5,20 +5,24 @@ namespace wf {
 namespace seq {
 
 template <typename T>
-__global__ void embed_f32_kernel(const T* __restrict__ table, const int32_t* __restrict__ tokens, int W, float* __restrict__ x, float scale, T* __restrict__ x_t) {
+__global__ void embed_f32_kernel(const T* __restrict__ table, const int32_t* __restrict__ tokens, int W, float* __restrict__ x, float scale, T* __restrict__ x_t,
+                                 const T* __restrict__ pos_table, const int32_t* __restrict__ tok_pos) {
     const int i = blockIdx.x;
     const T* row = table + (size_t)tokens[i] * W;
+    const T* prow = pos_table ? pos_table + (size_t)tok_pos[i] * W : nullptr;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float v = to_f(row[c]) * scale;
+        float v = to_f(row[c]) * scale;
+        if (prow) v += to_f(prow[c]);
         x[(size_t)i * W + c] = v;
         if (x_t) x_t[(size_t)i * W + c] = from_f<T>(v);
     }
 }
 
-int launch_embed_f32(int dt, const void* table, const int32_t* tokens, int n, int W, float* x, cudaStream_t s, float scale, void* x_t) {
+int launch_embed_f32(int dt, const void* table, const int32_t* tokens, int n, int W, float* x, cudaStream_t s, float scale, void* x_t,
+                     const void* pos_table, const int32_t* tok_pos) {
     if (n <= 0) return WF_OK;
-    if (dt == WF_BF16) embed_f32_kernel<<<n, 256, 0, s>>>((const __nv_bfloat16*)table, tokens, W, x, scale, (__nv_bfloat16*)x_t);
-    else embed_f32_kernel<<<n, 256, 0, s>>>((const float*)table, tokens, W, x, scale, (float*)x_t);
+    if (dt == WF_BF16) embed_f32_kernel<<<n, 256, 0, s>>>((const __nv_bfloat16*)table, tokens, W, x, scale, (__nv_bfloat16*)x_t, (const __nv_bfloat16*)pos_table, tok_pos);
+    else embed_f32_kernel<<<n, 256, 0, s>>>((const float*)table, tokens, W, x, scale, (float*)x_t, (const float*)pos_table, tok_pos);
     return launch_check(cudaGetLastError(), "embed_f32");
 }
 
@@ -211,6 +215,142 @@ int launch_add_dual_norm(int dt, float* x, const float* y1, float a1, const floa
     if (dt == WF_BF16) add_dual_norm_kernel<<<n, AD_THREADS, 0, s>>>(x, y1, a1, y2, a2, y3, (const __nv_bfloat16*)w1, (const __nv_bfloat16*)w2, w_offset, eps, W, (__nv_bfloat16*)h1, (__nv_bfloat16*)h2);
     else add_dual_norm_kernel<<<n, AD_THREADS, 0, s>>>(x, y1, a1, y2, a2, y3, (const float*)w1, (const float*)w2, w_offset, eps, W, (float*)h1, (float*)h2);
     return launch_check(cudaGetLastError(), "add_dual_norm");
+}
+
+// sum over the block of the squared distances from the mean, the row's values in keep (up to PER per thread) and in row (read beyond those)
+template <int PER>
+__device__ __forceinline__ float block_sq_dev(const float (&keep)[PER], const float* row, int W, float mean, float* scratch) {
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        if (c < W) { const float d = keep[k] - mean; ss = fmaf(d, d, ss); }
+    }
+    for (int c = threadIdx.x + PER * blockDim.x; c < W; c += blockDim.x) { const float d = row[c] - mean; ss = fmaf(d, d, ss); }
+    return block_sum(ss, scratch);
+}
+
+// one block per row; the row stays in registers between the two statistics and the store (re-read beyond LN_PER values per thread)
+constexpr int LN_PER = 8;
+template <typename T>
+__global__ void __launch_bounds__(512) layer_norm_kernel(const float* __restrict__ x, int ldx, const T* __restrict__ w, const T* __restrict__ b, float eps, int W,
+                                                         float* __restrict__ y, int ldy, T* __restrict__ y_t, int ldt, const int32_t* __restrict__ rows) {
+    __shared__ float scratch[33];
+    const int i = blockIdx.x;
+    const float* row = x + (size_t)(rows ? rows[i] : i) * ldx;
+    float keep[LN_PER], sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < LN_PER; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        keep[k] = c < W ? row[c] : 0.f;
+        sum += keep[k];
+    }
+    for (int c = threadIdx.x + LN_PER * blockDim.x; c < W; c += blockDim.x) sum += row[c];
+    const float mean = block_sum(sum, scratch) / (float)W;
+    const float inv = 1.f / sqrtf(block_sq_dev(keep, row, W, mean, scratch) / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < LN_PER; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        if (c >= W) continue;
+        const float v = (keep[k] - mean) * inv * to_f(w[c]) + to_f(b[c]);
+        if (y) y[(size_t)i * ldy + c] = v;
+        if (y_t) y_t[(size_t)i * ldt + c] = from_f<T>(v);
+    }
+    for (int c = threadIdx.x + LN_PER * blockDim.x; c < W; c += blockDim.x) {
+        const float v = (row[c] - mean) * inv * to_f(w[c]) + to_f(b[c]);
+        if (y) y[(size_t)i * ldy + c] = v;
+        if (y_t) y_t[(size_t)i * ldt + c] = from_f<T>(v);
+    }
+}
+
+int row_threads(int W) { return W > 1024 ? 512 : (W > 256 ? 256 : 128); }
+
+int launch_layer_norm(int dt, const float* x, int ldx, const void* w, const void* b, float eps, int n, int W, float* y, int ldy, void* y_t, int ldt,
+                      const int32_t* rows, cudaStream_t s) {
+    if (n <= 0) return WF_OK;
+    if (dt == WF_BF16) layer_norm_kernel<<<n, row_threads(W), 0, s>>>(x, ldx, (const __nv_bfloat16*)w, (const __nv_bfloat16*)b, eps, W, y, ldy, (__nv_bfloat16*)y_t, ldt, rows);
+    else layer_norm_kernel<<<n, row_threads(W), 0, s>>>(x, ldx, (const float*)w, (const float*)b, eps, W, y, ldy, (float*)y_t, ldt, rows);
+    return launch_check(cudaGetLastError(), "layer_norm");
+}
+
+// one block per row (launch_branch_add_norm)
+template <typename T>
+__global__ void __launch_bounds__(512) branch_add_norm_kernel(float* __restrict__ x, BranchSum bs, const T* __restrict__ w, const T* __restrict__ b, float w_offset, float eps,
+                                                              int W, T* __restrict__ h) {
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * W;
+    float* row = x + base;
+    const float* y1 = bs.y1 ? bs.y1 + base : nullptr;
+    const float* y2 = bs.y2 ? bs.y2 + base : nullptr;
+    const float* y3 = bs.y3 ? bs.y3 + base : nullptr;
+    const float* gate = bs.gate ? bs.gate + (size_t)blockIdx.x * bs.ldg : nullptr;
+    const T *pw1 = (const T*)bs.pw1, *pw2 = (const T*)bs.pw2, *gb1 = (const T*)bs.gb1, *gb2 = (const T*)bs.gb2;
+    float k1[LN_PER], k2[LN_PER];                  // the pair's outputs stay in registers between their norms and the sum
+    float f1 = bs.a1, f2 = bs.a2;
+#pragma unroll
+    for (int k = 0; k < LN_PER; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        k1[k] = y1 && c < W ? y1[c] : 0.f;
+        k2[k] = y2 && c < W ? y2[c] : 0.f;
+    }
+    if (pw1 && y1) {
+        float s1 = 0.f, s2 = 0.f;
+#pragma unroll
+        for (int k = 0; k < LN_PER; ++k) { s1 = fmaf(k1[k], k1[k], s1); s2 = fmaf(k2[k], k2[k], s2); }
+        for (int c = threadIdx.x + LN_PER * blockDim.x; c < W; c += blockDim.x) { s1 = fmaf(y1[c], y1[c], s1); if (y2) s2 = fmaf(y2[c], y2[c], s2); }
+        f1 *= 1.f / sqrtf(block_sum(s1, scratch) / (float)W + eps);
+        if (y2) f2 *= 1.f / sqrtf(block_sum(s2, scratch) / (float)W + eps);
+    }
+    auto updated = [&](int c, float v1, float v2) {
+        float v = row[c];
+        if (y1) {
+            float m = f1 * v1 * (pw1 ? to_f(pw1[c]) : 1.f);
+            if (y2) m += f2 * v2 * (pw2 ? to_f(pw2[c]) : 1.f);
+            float t = gate ? sigmoid_f(gate[c] + to_f(gb1[c])) * m : m;
+            if (y3) t += gate ? sigmoid_f(gate[W + c] + to_f(gb2[c])) * y3[c] : y3[c];
+            v += t;
+            row[c] = v;
+        }
+        return v;
+    };
+    float keep[LN_PER], sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < LN_PER; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        keep[k] = c < W ? updated(c, k1[k], k2[k]) : 0.f;
+        sum += keep[k];
+    }
+    for (int c = threadIdx.x + LN_PER * blockDim.x; c < W; c += blockDim.x) sum += updated(c, y1 ? y1[c] : 0.f, y2 ? y2[c] : 0.f);
+    if (!w) return;
+    const float mean = b ? block_sum(sum, scratch) / (float)W : 0.f;
+    const float inv = 1.f / sqrtf(block_sq_dev(keep, row, W, mean, scratch) / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < LN_PER; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        if (c < W) h[base + c] = from_f<T>((keep[k] - mean) * inv * (w_offset + to_f(w[c])) + (b ? to_f(b[c]) : 0.f));
+    }
+    for (int c = threadIdx.x + LN_PER * blockDim.x; c < W; c += blockDim.x)
+        h[base + c] = from_f<T>((row[c] - mean) * inv * (w_offset + to_f(w[c])) + (b ? to_f(b[c]) : 0.f));
+}
+
+int launch_branch_add_norm(int dt, float* x, const BranchSum& bs, const void* w, const void* b, float w_offset, float eps, int n, int W, void* h, cudaStream_t s) {
+    if (n <= 0) return WF_OK;
+    if ((bs.y2 || bs.y3) && !bs.y1) { set_error("branch_add_norm: a second output without a first"); return WF_ERR_INVALID; }
+    if (bs.y2 && (bs.pw1 != nullptr) != (bs.pw2 != nullptr)) { set_error("branch_add_norm: both outputs of a pair are normed or none"); return WF_ERR_INVALID; }
+    if (dt == WF_BF16) branch_add_norm_kernel<<<n, row_threads(W), 0, s>>>(x, bs, (const __nv_bfloat16*)w, (const __nv_bfloat16*)b, w_offset, eps, W, (__nv_bfloat16*)h);
+    else branch_add_norm_kernel<<<n, row_threads(W), 0, s>>>(x, bs, (const float*)w, (const float*)b, w_offset, eps, W, (float*)h);
+    return launch_check(cudaGetLastError(), "branch_add_norm");
+}
+
+__global__ void softcap_kernel(float* __restrict__ z, size_t count, float cap) {
+    for (size_t k = (size_t)blockIdx.x * blockDim.x + threadIdx.x; k < count; k += (size_t)gridDim.x * blockDim.x) z[k] = cap * tanhf(z[k] / cap);
+}
+
+int launch_softcap(float* z, size_t count, float cap, cudaStream_t s) {
+    if (count == 0) return WF_OK;
+    const int blocks = (int)((count + 255) / 256 > 4096 ? 4096 : (count + 255) / 256);
+    softcap_kernel<<<blocks, 256, 0, s>>>(z, count, cap);
+    return launch_check(cudaGetLastError(), "softcap");
 }
 
 // thread per (token, channel)

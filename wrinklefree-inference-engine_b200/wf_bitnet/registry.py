@@ -21,6 +21,8 @@ _MODULES: Dict[str, str] = {
     "NukezenForCausalLM": "sglang.srt.models.nukezen",
     "Fivedra": "sglang.srt.models.fivedra",
     "FivedraForCausalLM": "sglang.srt.models.fivedra",
+    "Fuvavik": "sglang.srt.models.fuvavik",
+    "FuvavikForCausalLM": "sglang.srt.models.fuvavik",
 }
 
 

@@ -99,6 +99,9 @@ class Scheduler:
     def add(self, req: Request) -> None:
         if not req.prompt:
             raise ValueError("empty prompt")
+        longest = int(getattr(self.model, "max_positions", 0))          # models with a table of positions end where it ends
+        if longest and len(req.prompt) + req.max_new_tokens - 1 > longest:      # the last drawn token is not fed back
+            raise ValueError(f"request {req.rid!r} needs {len(req.prompt) + req.max_new_tokens - 1} positions, the model has {longest}")
         self.waiting.append(req)
 
     def _admit(self) -> None:

@@ -49,6 +49,7 @@ class SeqCausalLM:
         self.native_config = nc
         self.engine = SeqEngine(nc, layers, build=build)
         self.vocab = c.vocab
+        self.max_positions = int(nc.max_positions)   # 0: no limit of the model's own
         self.max_step_tokens = max_step_tokens
 
     @classmethod
