@@ -1,14 +1,619 @@
-// Tensor-core forms of attention with mixed heads: not built yet, every shape takes the plain kernel (seq_attn.cu).
+// Grouped-query attention with mixed heads on tensor cores (bf16 mma.sync.m16n8k16, float softmax): head h applies
+// sum_g T[h, g] * (head g's softmax weights) to the values of its own key/value head, so every head of a token runs in one CTA.  Scores are
+// kept in units of log 2; the logarithmic distance penalty is r1 log2(1 + r2 distance) there.  Weights enter the value product as a two-term
+// bf16 split (as in seq_attn_mma.cu).
+//
+//   * prompt form (talk_prompt_kernel): a CTA takes up to 256 rows (token, head) of one sequence and walks the keys twice.  The first walk
+//     leaves every row's log-sum-exp (sink included) in registers; the second forms the normalised weights, mixes them across heads through
+//     shared memory in float and multiplies them with the values.  The mixture needs normalised weights of all heads at once, which is why
+//     one online pass does not do; with G key/value heads, the pass that keeps every head's weights apart (below) would cost G value products.
+//   * decode form (talk_decode_kernel, every sequence brings one token): few rows and a long key range, so the keys are read ONCE: the
+//     mixture being linear, every head's unmixed weights are applied to every key/value head's values, partial sums of the key splits go to a
+//     workspace, and talk_merge_kernel normalises and mixes them.
 #include "seq_attn_mma.cuh"
+#include <math.h>
+#include <algorithm>
 
 namespace wf {
 namespace seq {
 
-bool talk_attn_mma_usable(const GqaDims&, const PagedCache&) { return false; }
-size_t talk_attn_workspace(const GqaDims&, int, int) { return 0; }
-int launch_talk_attn_mma(const Batch&, const GqaDims&, const void*, const PagedCache&, void*, float*, int, cudaStream_t) {
-    set_error("attention: no tensor-core form with mixed heads");
-    return WF_ERR_UNSUPPORTED;
+namespace {
+
+constexpr int TK_THREADS = 256, TK_WARPS = 8;
+constexpr int TK_MAX_HEADS = 32, TK_UNITS = 16;      // heads; 16-row units per prompt CTA (two per warp)
+
+struct TalkParams {
+    int ub, rp2, rp2_log, tq;    // prompt form: units per key/value head, rows per token (group size rounded up to a power of two), tokens per CTA
+    int kt, nst;                 // decode form: keys per tile, staged tiles
+    int splits;
+    float* part;                 // decode form: [n][splits] of { [H][G][dv] weighted values, [H] maximum, [H] sum }
+};
+
+__host__ __device__ inline size_t talk_part_floats(const GqaDims& D) { return (size_t)D.H * D.G * D.dv + 2 * D.H; }
+
+// acc.{x,y} += p.{x,y} * t
+__device__ __forceinline__ void fma_x2(unsigned long long& acc, unsigned long long p, float t) {
+    unsigned long long tt;
+    asm("mov.b64 %0, {%1, %1};" : "=l"(tt) : "f"(t));
+    asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(acc) : "l"(p), "l"(tt));
+}
+__device__ __forceinline__ unsigned long long pack_x2(float a, float b) {
+    unsigned long long v;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(v) : "f"(a), "f"(b));
+    return v;
+}
+__device__ __forceinline__ void unpack_x2(unsigned long long v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+
+// two-term bf16 split of a pair: hi = round(a, b), lo = round(rest)
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const float ah = __bfloat162float(__float2bfloat16_rn(a)), bh = __bfloat162float(__float2bfloat16_rn(b));
+    hi = pack_bf16(ah, bh);
+    lo = pack_bf16(a - ah, b - bh);
+}
+
+// one tile of keys (or values) of every key/value head, rows padded with zeros to `dp` entries: dst [G][kt][dp + 8]
+__device__ __forceinline__ void stage_rows(const Batch& b, const GqaDims& D, const PagedCache& pc, const int32_t* bt, uint32_t dst, size_t base, int d, int dp, int kt, int j0,
+                                           int pos_last) {
+    const int kc = dp / 8, rstep = TK_THREADS / kc, part = threadIdx.x % kc, row0 = threadIdx.x / kc;
+    if (row0 >= rstep) return;
+    const bool col_ok = part * 8 < d;
+    const int stride = dp + 8;
+    for (int key = row0; key < kt; key += rstep) {
+        const int j = j0 + key;
+        const bool ok = j <= pos_last;
+        const int jj = ok ? j : 0, pg = jj / pc.page_size, slot = jj - pg * pc.page_size;
+        const __nv_bfloat16* src = (const __nv_bfloat16*)pc.pool + (size_t)bt[pg] * pc.page_stride + pc.layer_off + base + (size_t)slot * d + (col_ok ? part * 8 : 0);
+        for (int g = 0; g < D.G; ++g) am_cp16(dst + (uint32_t)((g * kt + key) * stride + part * 8) * 2u, src + (size_t)g * pc.page_size * d, ok && col_ok);
+    }
+}
+
+// ---- prompt form --------------------------------------------------------------------------------------------------------------------
+template <int DKP, int DVP, int KT>
+struct TalkPromptShared {
+    static constexpr int KS = DKP + 8, VS = DVP + 8, XS = KS > VS ? KS : VS;      // row strides in elements
+    static constexpr int PS = KT + 4, WS = KT + 8;                                 // weights: floats, bf16
+    static size_t bytes(int G, int units, int H) {
+        const int hp = (H + 7) / 8 * 8;
+        return (size_t)2 * G * KT * XS * 2 + (size_t)units * 16 * (PS * 4 + 2 * WS * 2) + (size_t)H * hp * 4;
+    }
+};
+
+template <int DKP, int DVP, int KT>
+__global__ void __launch_bounds__(TK_THREADS, 1) talk_prompt_kernel(Batch b, GqaDims D, const __nv_bfloat16* __restrict__ qn, PagedCache pc, __nv_bfloat16* __restrict__ out,
+                                                                    TalkParams tp) {
+    using SH = TalkPromptShared<DKP, DVP, KT>;
+    constexpr int KS = SH::KS, VS = SH::VS, PS = SH::PS, WS = SH::WS, NKS = DKP / 16, NVT = DVP / 8, NST = KT / 8;
+    extern __shared__ __align__(16) unsigned char smraw[];
+    const int units = D.G * tp.ub, rows = units * 16, hp = (D.H + 7) / 8 * 8;
+    __nv_bfloat16* buf0 = reinterpret_cast<__nv_bfloat16*>(smraw);                 // keys (first walk: even tiles)
+    __nv_bfloat16* buf1 = buf0 + (size_t)D.G * KT * SH::XS;                        // values (first walk: keys of odd tiles)
+    float* P = reinterpret_cast<float*>(buf1 + (size_t)D.G * KT * SH::XS);         // [rows][PS] normalised weights
+    __nv_bfloat16* Wh = reinterpret_cast<__nv_bfloat16*>(P + (size_t)rows * PS);   // [rows][WS] mixed weights, high and low terms
+    __nv_bfloat16* Wl = Wh + (size_t)rows * WS;
+    float* Tt = reinterpret_cast<float*>(Wl + (size_t)rows * WS);                  // [H][hp]: Tt[g][h] = T[h, g]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3, rep = D.H / D.G;
+    int sq = -1, tok0 = 0, ntok = 0;
+    {
+        int t = (int)(gridDim.x - 1 - blockIdx.x);         // the last tiles of a sequence see the most keys: they start first
+        for (int s = 0; s < b.nseq; ++s) {
+            const int tiles = (b.seq_len[s] + tp.tq - 1) / tp.tq;
+            if (t < tiles) { sq = s; tok0 = t * tp.tq; ntok = b.seq_len[s] - tok0 < tp.tq ? b.seq_len[s] - tok0 : tp.tq; break; }
+            t -= tiles;
+        }
+    }
+    if (sq < 0) return;
+    const int flat0 = b.seq_start[sq] + tok0, pos0 = b.seq_pos0[sq] + tok0, pos_last = pos0 + ntok - 1;
+    const int32_t* bt = pc.block_table + (size_t)b.seq_slot[sq] * pc.max_blocks;
+    for (int e = tid; e < D.H * hp; e += TK_THREADS) { const int g = e / hp, h = e - g * hp; Tt[e] = h < D.H ? D.talk[h * D.H + g] : 0.f; }
+    // the warp's units: 16 rows each, row r of unit u -> key/value head u / ub, row (u % ub) * 16 + r of that head -> token, head of the group
+    bool r_ok[2][2];
+    int r_pos[2][2], r_lo[2][2], r_kv[2], r_tok[2][2], r_head[2][2];
+    float r_lse[2][2], r_r1[2][2], r_r2[2][2];
+    uint32_t qf[2][NKS][4];
+#pragma unroll
+    for (int un = 0; un < 2; ++un) {
+        const int u = warp + un * TK_WARPS, kv = u < units ? u / tp.ub : 0, base = (u - kv * tp.ub) * 16;
+        r_kv[un] = kv;
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int r = base + g4 + 8 * k, tk = r >> tp.rp2_log, hg = r & (tp.rp2 - 1);
+            r_ok[un][k] = u < units && tk < ntok && hg < rep;
+            r_tok[un][k] = flat0 + (r_ok[un][k] ? tk : 0); r_head[un][k] = kv * rep + (r_ok[un][k] ? hg : 0);
+            r_pos[un][k] = pos0 + (r_ok[un][k] ? tk : 0);
+            int lo = r_pos[un][k] - D.window + 1;
+            if (D.chunk > 0) { const int c0 = r_pos[un][k] / D.chunk * D.chunk; if (c0 > lo) lo = c0; }
+            r_lo[un][k] = lo;
+            r_r1[un][k] = D.dist_r1 ? D.dist_r1[r_head[un][k]] : 0.f;
+            r_r2[un][k] = D.dist_r1 ? D.dist_r2[r_head[un][k]] : 0.f;
+            const __nv_bfloat16* q = qn + ((size_t)r_tok[un][k] * D.H + r_head[un][k]) * D.d;
+#pragma unroll
+            for (int ks = 0; ks < NKS; ++ks)
+#pragma unroll
+                for (int hlf = 0; hlf < 2; ++hlf) {
+                    const int c = ks * 16 + hlf * 8 + 2 * t4;
+                    qf[un][ks][k + 2 * hlf] = r_ok[un][k] && c < D.d ? *reinterpret_cast<const uint32_t*>(q + c) : 0u;
+                }
+        }
+    }
+    const float scale2 = D.scale * LOG2E;
+    int lo_all = pos0 - D.window + 1 > 0 ? pos0 - D.window + 1 : 0;
+    if (D.chunk > 0) { const int c0 = pos0 / D.chunk * D.chunk; if (c0 > lo_all) lo_all = c0; }
+    const int t_lo = lo_all / KT, t_hi = pos_last / KT;
+    const uint32_t sb0 = smem_u32(buf0), sb1 = smem_u32(buf1);
+    const size_t v_base = (size_t)D.G * pc.page_size * D.d;
+    const int mi = lane >> 3, rr = lane & 7;
+    // scores of one unit on the tile at kb whose first key is j0: penalised, masked, units of log 2
+    auto unit_scores = [&](int un, uint32_t kb, int j0, float (&s)[NST][4]) {
+#pragma unroll
+        for (int j = 0; j < NST; ++j) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
+        const uint32_t kbu = kb + (uint32_t)(r_kv[un] * KT * KS) * 2u;
+#pragma unroll
+        for (int ks = 0; ks < NKS; ++ks)
+#pragma unroll
+            for (int jp = 0; jp < NST / 2; ++jp) {
+                uint32_t kf[4];
+                am_ldsm_x4(kf, kbu + (uint32_t)((jp * 16 + (mi >> 1) * 8 + rr) * KS + ks * 16 + (mi & 1) * 8) * 2u);
+                am_mma(s[2 * jp], qf[un][ks], kf[0], kf[1]);
+                am_mma(s[2 * jp + 1], qf[un][ks], kf[2], kf[3]);
+            }
+#pragma unroll
+        for (int j = 0; j < NST; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int k = e >> 1, key = j0 + j * 8 + 2 * t4 + (e & 1), dist = r_pos[un][k] - key;
+                const float pen = r_r1[un][k] * __log2f(fmaf(r_r2[un][k], (float)max(dist, 0), 1.f));
+                s[j][e] = r_ok[un][k] && dist >= 0 && key >= r_lo[un][k] ? fmaf(s[j][e], scale2, -pen) : -INFINITY;
+            }
+    };
+    // ---- first walk: log-sum-exp of every row
+    {
+        float m_run[2][2] = {{-INFINITY, -INFINITY}, {-INFINITY, -INFINITY}}, l_run[2][2] = {{0.f, 0.f}, {0.f, 0.f}};
+        stage_rows(b, D, pc, bt, sb0, 0, D.d, DKP, KT, t_lo * KT, pos_last);
+        am_commit();
+        for (int t = t_lo; t <= t_hi; ++t) {
+            am_wait<0>();
+            __syncthreads();
+            if (t < t_hi) { stage_rows(b, D, pc, bt, (t - t_lo) & 1 ? sb0 : sb1, 0, D.d, DKP, KT, (t + 1) * KT, pos_last); am_commit(); }
+            const uint32_t kb = (t - t_lo) & 1 ? sb1 : sb0;
+#pragma unroll
+            for (int un = 0; un < 2; ++un) {
+                if (warp + un * TK_WARPS >= units) continue;
+                float s[NST][4];
+                unit_scores(un, kb, t * KT, s);
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {
+                    float mx = -INFINITY;
+#pragma unroll
+                    for (int j = 0; j < NST; ++j) mx = fmaxf(mx, fmaxf(s[j][2 * k], s[j][2 * k + 1]));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+                    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+                    const float mn = fmaxf(m_run[un][k], mx), ms = mn == -INFINITY ? 0.f : mn;
+                    float ls = 0.f;
+#pragma unroll
+                    for (int j = 0; j < NST; ++j) ls += exp2f(s[j][2 * k] - ms) + exp2f(s[j][2 * k + 1] - ms);
+                    l_run[un][k] = l_run[un][k] * exp2f(m_run[un][k] - ms) + ls;      // nothing seen yet: exp2(-inf) = 0
+                    m_run[un][k] = mn;
+                }
+            }
+        }
+#pragma unroll
+        for (int un = 0; un < 2; ++un)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                float l = l_run[un][k];
+                l += __shfl_xor_sync(0xffffffffu, l, 1);
+                l += __shfl_xor_sync(0xffffffffu, l, 2);
+                // weights are exp2(score - lse): -log2 of what a weight 2^m would be multiplied by, the sink's share included
+                r_lse[un][k] = r_ok[un][k] ? m_run[un][k] - log2f(am_inv_sum(D, r_head[un][k], m_run[un][k], l)) : 0.f;
+            }
+        __syncthreads();                                   // both buffers are free
+    }
+    // ---- second walk: weights, mixture, values
+    float o[2][NVT][4];
+#pragma unroll
+    for (int un = 0; un < 2; ++un)
+#pragma unroll
+        for (int j = 0; j < NVT; ++j) { o[un][j][0] = o[un][j][1] = o[un][j][2] = o[un][j][3] = 0.f; }
+    stage_rows(b, D, pc, bt, sb0, 0, D.d, DKP, KT, t_lo * KT, pos_last);
+    am_commit();
+    const uint32_t wh = smem_u32(Wh), wl = smem_u32(Wl);
+    const int jq_n = KT / 4, mix_items = (hp / 8) * tp.tq * jq_n;
+    for (int t = t_lo; t <= t_hi; ++t) {
+        am_wait<0>();
+        __syncthreads();                                   // the keys are there; everyone is done with the values and the mixed weights
+        stage_rows(b, D, pc, bt, sb1, v_base, D.dv, DVP, KT, t * KT, pos_last);
+        am_commit();
+#pragma unroll
+        for (int un = 0; un < 2; ++un) {
+            const int u = warp + un * TK_WARPS;
+            if (u >= units) continue;
+            float s[NST][4];
+            unit_scores(un, sb0, t * KT, s);
+#pragma unroll
+            for (int j = 0; j < NST; ++j)
+#pragma unroll
+                for (int k = 0; k < 2; ++k)
+                    *reinterpret_cast<float2*>(P + (size_t)(u * 16 + g4 + 8 * k) * PS + j * 8 + 2 * t4) =
+                        make_float2(exp2f(s[j][2 * k] - r_lse[un][k]), exp2f(s[j][2 * k + 1] - r_lse[un][k]));
+        }
+        __syncthreads();                                   // every head's weights are there; the keys are free
+        if (t < t_hi) stage_rows(b, D, pc, bt, sb0, 0, D.d, DKP, KT, (t + 1) * KT, pos_last);
+        am_commit();
+        for (int it = tid; it < mix_items; it += TK_THREADS) {         // eight heads of a token on four keys
+            const int jq = it % jq_n, tk = (it / jq_n) % tp.tq, hb = it / (jq_n * tp.tq);
+            unsigned long long acc[8][2];
+#pragma unroll
+            for (int h = 0; h < 8; ++h) acc[h][0] = acc[h][1] = 0ull;
+            const float* pr = P + (size_t)(tk << tp.rp2_log) * PS + jq * 4;
+            const float* tr = Tt + hb * 8;
+            for (int kv = 0; kv < D.G; ++kv, pr += (size_t)tp.ub * 16 * PS) {
+                for (int hg = 0; hg < rep; ++hg, tr += hp) {
+                    const float4 p = *reinterpret_cast<const float4*>(pr + hg * PS);
+                    const float4 ta = *reinterpret_cast<const float4*>(tr), tb = *reinterpret_cast<const float4*>(tr + 4);
+                    const unsigned long long p0 = pack_x2(p.x, p.y), p1 = pack_x2(p.z, p.w);
+                    fma_x2(acc[0][0], p0, ta.x); fma_x2(acc[0][1], p1, ta.x); fma_x2(acc[1][0], p0, ta.y); fma_x2(acc[1][1], p1, ta.y);
+                    fma_x2(acc[2][0], p0, ta.z); fma_x2(acc[2][1], p1, ta.z); fma_x2(acc[3][0], p0, ta.w); fma_x2(acc[3][1], p1, ta.w);
+                    fma_x2(acc[4][0], p0, tb.x); fma_x2(acc[4][1], p1, tb.x); fma_x2(acc[5][0], p0, tb.y); fma_x2(acc[5][1], p1, tb.y);
+                    fma_x2(acc[6][0], p0, tb.z); fma_x2(acc[6][1], p1, tb.z); fma_x2(acc[7][0], p0, tb.w); fma_x2(acc[7][1], p1, tb.w);
+                }
+            }
+#pragma unroll
+            for (int h8 = 0; h8 < 8; ++h8) {
+                const int h = hb * 8 + h8;
+                if (h >= D.H) break;
+                float a, c, e, f;
+                unpack_x2(acc[h8][0], a, c);
+                unpack_x2(acc[h8][1], e, f);
+                uint2 hi, lo;
+                split_pair(a, c, hi.x, lo.x);
+                split_pair(e, f, hi.y, lo.y);
+                const size_t at = (size_t)((h / rep) * tp.ub * 16 + (tk << tp.rp2_log) + h % rep) * WS + jq * 4;
+                *reinterpret_cast<uint2*>(Wh + at) = hi;
+                *reinterpret_cast<uint2*>(Wl + at) = lo;
+            }
+        }
+        am_wait<1>();
+        __syncthreads();                                   // mixed weights and values are there
+#pragma unroll
+        for (int un = 0; un < 2; ++un) {
+            const int u = warp + un * TK_WARPS;
+            if (u >= units) continue;
+            const uint32_t vb = sb1 + (uint32_t)(r_kv[un] * KT * VS) * 2u;
+#pragma unroll
+            for (int kk = 0; kk < KT / 16; ++kk) {
+                uint32_t ph[4], pl[4];
+                const uint32_t at = (uint32_t)((u * 16 + (lane & 15)) * WS + kk * 16 + (lane >> 4) * 8) * 2u;
+                am_ldsm_x4(ph, wh + at);
+                am_ldsm_x4(pl, wl + at);
+#pragma unroll
+                for (int np = 0; np < NVT / 2; ++np) {
+                    uint32_t vf[4];
+                    am_ldsm_x4_trans(vf, vb + (uint32_t)((kk * 16 + (mi & 1) * 8 + rr) * VS + np * 16 + (mi >> 1) * 8) * 2u);
+                    am_mma(o[un][2 * np], ph, vf[0], vf[1]);
+                    am_mma(o[un][2 * np], pl, vf[0], vf[1]);
+                    am_mma(o[un][2 * np + 1], ph, vf[2], vf[3]);
+                    am_mma(o[un][2 * np + 1], pl, vf[2], vf[3]);
+                }
+            }
+        }
+    }
+    am_wait<0>();
+#pragma unroll
+    for (int un = 0; un < 2; ++un)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            if (!r_ok[un][k]) continue;
+            __nv_bfloat16* dst = out + ((size_t)r_tok[un][k] * D.H + r_head[un][k]) * D.dv;
+#pragma unroll
+            for (int j = 0; j < NVT; ++j) {
+                const int c = j * 8 + 2 * t4;
+                if (c < D.dv) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[un][j][2 * k], o[un][j][2 * k + 1]);
+            }
+        }
+}
+
+// ---- decode form --------------------------------------------------------------------------------------------------------------------
+// shared memory of the decode form, in order: keys [nst][G][kt][kp + 8], values [nst][G][kt][vp + 8], queries [G][rp][kp + 8] (all bf16; kp,
+// vp: sizes rounded up to 16, rp: group size rounded up to 8), scores float [H][kt + 4], weights bf16 [2][16 MT][kt + 8], maximum, sum and
+// correction float [3][H]
+struct TalkDecodeShared {
+    int kp, vp, rp, mt;
+    size_t k_tile, v_tile, q, sc, w;
+    __host__ __device__ TalkDecodeShared(const GqaDims& D, int kt) {
+        kp = (D.d + 15) / 16 * 16; vp = (D.dv + 15) / 16 * 16; rp = (D.H / D.G + 7) / 8 * 8; mt = (D.H + 15) / 16;
+        k_tile = (size_t)D.G * kt * (kp + 8) * 2; v_tile = (size_t)D.G * kt * (vp + 8) * 2; q = (size_t)D.G * rp * (kp + 8) * 2;
+        sc = (size_t)D.H * (kt + 4) * 4; w = (size_t)mt * 16 * (kt + 8) * 2;
+    }
+    __host__ __device__ size_t bytes(const GqaDims& D, int nst) const { return nst * (k_tile + v_tile) + q + sc + 2 * w + (size_t)3 * D.H * 4; }
+};
+
+// MT: 16-row tiles of heads; IT: (key/value head, 16 value columns) items per warp
+template <int MT, int IT>
+__global__ void __launch_bounds__(TK_THREADS, MT * IT <= 10 ? 2 : 1) talk_decode_kernel(Batch b, GqaDims D, const __nv_bfloat16* __restrict__ qn, PagedCache pc, TalkParams tp) {
+    extern __shared__ __align__(16) unsigned char smraw[];
+    const TalkDecodeShared sh(D, tp.kt);
+    const int KT = tp.kt, KS = sh.kp + 8, VS = sh.vp + 8, SS = KT + 4, WS = KT + 8, nks = sh.kp / 16, rep = D.H / D.G;
+    unsigned char* ks_ = smraw;
+    unsigned char* vs_ = ks_ + tp.nst * sh.k_tile;
+    __nv_bfloat16* Q = reinterpret_cast<__nv_bfloat16*>(vs_ + tp.nst * sh.v_tile);
+    float* Sc = reinterpret_cast<float*>(reinterpret_cast<unsigned char*>(Q) + sh.q);
+    __nv_bfloat16* Wh = reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<unsigned char*>(Sc) + sh.sc);
+    __nv_bfloat16* Wl = reinterpret_cast<__nv_bfloat16*>(reinterpret_cast<unsigned char*>(Wh) + sh.w);
+    float* hm = reinterpret_cast<float*>(reinterpret_cast<unsigned char*>(Wl) + sh.w);
+    float *hl = hm + D.H, *hc = hl + D.H;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3, mi = lane >> 3, rr = lane & 7;
+    const int sq = blockIdx.x, split = blockIdx.y, tok = b.seq_start[sq], pos = b.seq_pos0[sq];
+    const int32_t* bt = pc.block_table + (size_t)b.seq_slot[sq] * pc.max_blocks;
+    int lo = pos - D.window + 1 > 0 ? pos - D.window + 1 : 0;
+    if (D.chunk > 0) { const int c0 = pos / D.chunk * D.chunk; if (c0 > lo) lo = c0; }
+    int t_lo = lo / KT, t_hi = pos / KT;
+    {
+        const int per = (t_hi - t_lo + tp.splits) / tp.splits;
+        t_lo += split * per;
+        if (t_lo + per - 1 < t_hi) t_hi = t_lo + per - 1;
+    }
+    const size_t v_base = (size_t)D.G * pc.page_size * D.d;
+    const uint32_t sk = smem_u32(ks_), sv = smem_u32(vs_), sq_ = smem_u32(Q), wh = smem_u32(Wh), wl = smem_u32(Wl);
+    auto stage = [&](int t, int bf) {
+        stage_rows(b, D, pc, bt, sk + (uint32_t)(bf * sh.k_tile), 0, D.d, sh.kp, KT, t * KT, pos);
+        stage_rows(b, D, pc, bt, sv + (uint32_t)(bf * sh.v_tile), v_base, D.dv, sh.vp, KT, t * KT, pos);
+        am_commit();
+    };
+    if (tp.nst == 2 && t_lo <= t_hi) stage(t_lo, 0);
+    for (int e = tid; e < D.G * sh.rp * sh.kp; e += TK_THREADS) {
+        const int r = e / sh.kp, c = e - r * sh.kp, kv = r / sh.rp, hg = r - kv * sh.rp;
+        Q[r * KS + c] = hg < rep && c < D.d ? qn[((size_t)tok * D.H + kv * rep + hg) * D.d + c] : __float2bfloat16_rn(0.f);
+    }
+    for (int e = tid; e < (MT * 16 - D.H) * WS; e += TK_THREADS) { Wh[D.H * WS + e] = __float2bfloat16_rn(0.f); Wl[D.H * WS + e] = __float2bfloat16_rn(0.f); }
+    for (int h = tid; h < D.H; h += TK_THREADS) { hm[h] = -INFINITY; hl[h] = 0.f; }
+    const float scale2 = D.scale * LOG2E;
+    const int nc = sh.vp / 16, items = D.G * nc;
+    float o[IT][MT][2][4];
+#pragma unroll
+    for (int i = 0; i < IT; ++i)
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int c = 0; c < 2; ++c) { o[i][m][c][0] = o[i][m][c][1] = o[i][m][c][2] = o[i][m][c][3] = 0.f; }
+    for (int t = t_lo; t <= t_hi; ++t) {
+        int bf = 0;
+        if (tp.nst == 2) {
+            bf = (t - t_lo) & 1;
+            am_wait<0>();
+            __syncthreads();                               // the tile is there; everyone is done with the other buffer
+            if (t < t_hi) stage(t + 1, bf ^ 1);
+        } else {
+            __syncthreads();
+            stage(t, 0);
+            am_wait<0>();
+            __syncthreads();
+        }
+        const uint32_t kb = sk + (uint32_t)(bf * sh.k_tile), vb = sv + (uint32_t)(bf * sh.v_tile);
+        // ---- raw scores, keys as the M rows and the heads of one key/value head as 8-wide N tiles
+        const int kgroups = KT / 16, nr = sh.rp / 8;
+        for (int it = warp; it < D.G * kgroups * nr; it += TK_WARPS) {
+            const int n8 = it % nr, kk = (it / nr) % kgroups, kv = it / (nr * kgroups);
+            float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            const uint32_t ka = kb + (uint32_t)((kv * KT + kk * 16 + (mi & 1) * 8 + rr) * KS + (mi >> 1) * 8) * 2u;
+            const uint32_t qa = sq_ + (uint32_t)((kv * sh.rp + n8 * 8 + rr) * KS + mi * 8) * 2u;
+            int ks = 0;
+            for (; ks + 1 < nks; ks += 2) {                // two k-steps per query load, two accumulation chains
+                uint32_t kf[4], kg[4], qf[4];
+                am_ldsm_x4(qf, qa + (uint32_t)ks * 32u);
+                am_ldsm_x4(kf, ka + (uint32_t)ks * 32u);
+                am_ldsm_x4(kg, ka + (uint32_t)ks * 32u + 32u);
+                am_mma(s[0], kf, qf[0], qf[1]);
+                am_mma(s[1], kg, qf[2], qf[3]);
+            }
+            if (ks < nks) {
+                uint32_t kf[4], qf[4];
+                am_ldsm_x4(qf, sq_ + (uint32_t)((kv * sh.rp + n8 * 8 + rr) * KS + ks * 16 + (mi & 1) * 8) * 2u);
+                am_ldsm_x4(kf, ka + (uint32_t)ks * 32u);
+                am_mma(s[0], kf, qf[0], qf[1]);
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int hg = n8 * 8 + 2 * t4 + (e & 1), key = kk * 16 + g4 + 8 * (e >> 1);
+                if (hg < rep) Sc[(kv * rep + hg) * SS + key] = s[0][e] + s[1][e];
+            }
+        }
+        __syncthreads();
+        // ---- online softmax, a warp per head, a lane per key
+        for (int h = warp; h < D.H; h += TK_WARPS) {
+            const int key = t * KT + lane, dist = pos - key;
+            float v = -INFINITY;
+            if (lane < KT && dist >= 0 && key >= lo) {
+                const float pen = D.dist_r1 ? D.dist_r1[h] * __log2f(fmaf(D.dist_r2[h], (float)dist, 1.f)) : 0.f;
+                v = fmaf(Sc[h * SS + lane], scale2, -pen);
+            }
+            const float mo = hm[h], mn = fmaxf(mo, warp_max(v)), ms = mn == -INFINITY ? 0.f : mn;
+            const float p = exp2f(v - ms), ls = warp_sum(p);
+            if (lane < KT) {
+                const __nv_bfloat16 ph = __float2bfloat16_rn(p);
+                Wh[h * WS + lane] = ph;
+                Wl[h * WS + lane] = __float2bfloat16_rn(p - __bfloat162float(ph));
+            }
+            __syncwarp();
+            if (lane == 0) { const float c = exp2f(mo - ms); hc[h] = c; hl[h] = hl[h] * c + ls; hm[h] = mn; }
+        }
+        __syncthreads();
+        // ---- every head's weights on every key/value head's values
+        float corr[MT][2];
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) { const int h = m * 16 + g4 + 8 * k; corr[m][k] = h < D.H ? hc[h] : 0.f; }
+#pragma unroll
+        for (int i = 0; i < IT; ++i)
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int c = 0; c < 2; ++c) { o[i][m][c][0] *= corr[m][0]; o[i][m][c][1] *= corr[m][0]; o[i][m][c][2] *= corr[m][1]; o[i][m][c][3] *= corr[m][1]; }
+        for (int kk = 0; kk < KT / 16; ++kk) {
+            uint32_t ph[MT][4], pl[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+                const uint32_t at = (uint32_t)((m * 16 + (lane & 15)) * WS + kk * 16 + (lane >> 4) * 8) * 2u;
+                am_ldsm_x4(ph[m], wh + at);
+                am_ldsm_x4(pl[m], wl + at);
+            }
+#pragma unroll
+            for (int i = 0; i < IT; ++i) {
+                const int it = warp + i * TK_WARPS;
+                if (it < items) {
+                    const int kv = it / nc, cc = it - kv * nc;
+                    uint32_t vf[4];
+                    am_ldsm_x4_trans(vf, vb + (uint32_t)((kv * KT + kk * 16 + (mi & 1) * 8 + rr) * VS + cc * 16 + (mi >> 1) * 8) * 2u);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        am_mma(o[i][m][0], ph[m], vf[0], vf[1]);
+                        am_mma(o[i][m][1], ph[m], vf[2], vf[3]);
+                        am_mma(o[i][m][0], pl[m], vf[0], vf[1]);
+                        am_mma(o[i][m][1], pl[m], vf[2], vf[3]);
+                    }
+                }
+            }
+        }
+    }
+    am_wait<0>();
+    float* part = tp.part + ((size_t)sq * tp.splits + split) * talk_part_floats(D);
+#pragma unroll
+    for (int i = 0; i < IT; ++i) {
+        const int it = warp + i * TK_WARPS;
+        if (it >= items) continue;
+        const int kv = it / nc, cc = it - kv * nc;
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) {
+                const int h = m * 16 + g4 + 8 * k;
+                if (h >= D.H) continue;
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    const int col = cc * 16 + c * 8 + 2 * t4;
+                    if (col < D.dv) *reinterpret_cast<float2*>(part + ((size_t)h * D.G + kv) * D.dv + col) = make_float2(o[i][m][c][2 * k], o[i][m][c][2 * k + 1]);
+                }
+            }
+    }
+    __syncthreads();
+    float* ml = part + (size_t)D.H * D.G * D.dv;
+    for (int h = tid; h < D.H; h += TK_THREADS) { ml[h] = hm[h]; ml[D.H + h] = hl[h]; }
+}
+
+// block per (token, head): normalise the source heads over the splits, mix, write.  blockDim = (values rounded up to 32, slices of the sum)
+__global__ void talk_merge_kernel(Batch b, GqaDims D, int splits, const float* __restrict__ parts, __nv_bfloat16* __restrict__ out) {
+    extern __shared__ float cf[];                          // [splits][H] factors, then [slices][dv] partial sums
+    const int sq = blockIdx.x, h = blockIdx.y, kv = h / (D.H / D.G), tok = b.seq_start[sq];
+    const int tid = threadIdx.y * blockDim.x + threadIdx.x;
+    const size_t pf = talk_part_floats(D), mo = (size_t)D.H * D.G * D.dv;
+    const float* p = parts + (size_t)sq * splits * pf;
+    float* red = cf + splits * D.H;
+    for (int g = tid; g < D.H; g += blockDim.x * blockDim.y) {
+        float m = -INFINITY, l = 0.f;
+        for (int s = 0; s < splits; ++s) m = fmaxf(m, p[s * pf + mo + g]);
+        for (int s = 0; s < splits; ++s) { const float f = exp2f(p[s * pf + mo + g] - m); cf[s * D.H + g] = f; l = fmaf(p[s * pf + mo + D.H + g], f, l); }
+        const float w = D.talk[h * D.H + g] * am_inv_sum(D, g, m, l);
+        for (int s = 0; s < splits; ++s) cf[s * D.H + g] *= w;
+    }
+    __syncthreads();
+    const int c = threadIdx.x;
+    float v = 0.f;
+    if (c < D.dv) {
+        const float* src = p + (size_t)kv * D.dv + c;
+        const int total = splits * D.H;
+#pragma unroll 4
+        for (int e = threadIdx.y; e < total; e += blockDim.y) { const int s = e / D.H, g = e - s * D.H; v = fmaf(cf[e], src[s * pf + (size_t)g * D.G * D.dv], v); }
+        red[threadIdx.y * D.dv + c] = v;
+    }
+    __syncthreads();
+    if (threadIdx.y == 0 && c < D.dv) {
+        for (int y = 1; y < (int)blockDim.y; ++y) v += red[y * D.dv + c];
+        out[((size_t)tok * D.H + h) * D.dv + c] = __float2bfloat16_rn(v);
+    }
+}
+
+constexpr size_t TK_SMEM = 227 * 1024 - 1024;
+
+int prompt_units(const GqaDims& D) { return std::max(1, TK_UNITS / D.G); }     // per key/value head
+
+// keys per tile of the prompt form (0: the sizes do not fit)
+int prompt_keys(const GqaDims& D) {
+    const int units = D.G * prompt_units(D);
+    if (units > TK_UNITS) return 0;
+    auto bytes = [&](int kt) {
+        const size_t x = std::max(D.d <= 64 ? 72 : 136, D.dv <= 64 ? 72 : 136);
+        const size_t hp = (D.H + 7) / 8 * 8;
+        return (size_t)4 * D.G * kt * x + (size_t)units * 16 * ((kt + 4) * 4 + (kt + 8) * 4) + D.H * hp * 4;
+    };
+    return bytes(32) <= TK_SMEM ? 32 : (bytes(16) <= TK_SMEM ? 16 : 0);
+}
+
+template <int DKP, int DVP, int KT>
+int prompt_launch(const Batch& b, const GqaDims& D, const void* qn, const PagedCache& pc, void* out, const TalkParams& tp, cudaStream_t s) {
+    const size_t smem = TalkPromptShared<DKP, DVP, KT>::bytes(D.G, D.G * tp.ub, D.H);
+    static DevOnce once;
+    if (once.need() && cuda_check(cudaFuncSetAttribute(talk_prompt_kernel<DKP, DVP, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TK_SMEM), "attention shared memory")) return WF_ERR_CUDA;
+    // every sequence's tokens are cut into tiles of tq; n / tq + nseq bounds their number (blocks beyond the last tile return at once)
+    talk_prompt_kernel<DKP, DVP, KT><<<b.n / tp.tq + b.nseq, TK_THREADS, smem, s>>>(b, D, (const __nv_bfloat16*)qn, pc, (__nv_bfloat16*)out, tp);
+    return launch_check(cudaGetLastError(), "talk_prompt");
+}
+
+template <int KT>
+int prompt_dispatch(const Batch& b, const GqaDims& D, const void* qn, const PagedCache& pc, void* out, const TalkParams& tp, cudaStream_t s) {
+    if (D.d <= 64) return D.dv <= 64 ? prompt_launch<64, 64, KT>(b, D, qn, pc, out, tp, s) : prompt_launch<64, 128, KT>(b, D, qn, pc, out, tp, s);
+    return D.dv <= 64 ? prompt_launch<128, 64, KT>(b, D, qn, pc, out, tp, s) : prompt_launch<128, 128, KT>(b, D, qn, pc, out, tp, s);
+}
+
+// tile and ring depth of the decode form; false where the accumulators or the tiles do not fit
+bool decode_shape(const GqaDims& D, int& kt, int& nst) {
+    const int mt = (D.H + 15) / 16, items = D.G * ((D.dv + 15) / 16), it = (items + TK_WARPS - 1) / TK_WARPS;
+    if (mt > 2 || it > (mt == 1 ? 16 : 8)) return false;
+    const int shapes[3][2] = {{32, 2}, {16, 2}, {16, 1}};
+    for (const auto& x : shapes)
+        if (TalkDecodeShared(D, x[0]).bytes(D, x[1]) <= TK_SMEM) { kt = x[0]; nst = x[1]; return true; }
+    return false;
+}
+
+template <int MT, int IT>
+int decode_launch(const Batch& b, const GqaDims& D, const void* qn, const PagedCache& pc, const TalkParams& tp, cudaStream_t s) {
+    static DevOnce once;
+    if (once.need() && cuda_check(cudaFuncSetAttribute(talk_decode_kernel<MT, IT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TK_SMEM), "attention shared memory")) return WF_ERR_CUDA;
+    talk_decode_kernel<MT, IT><<<dim3(b.nseq, tp.splits), TK_THREADS, TalkDecodeShared(D, tp.kt).bytes(D, tp.nst), s>>>(b, D, (const __nv_bfloat16*)qn, pc, tp);
+    return launch_check(cudaGetLastError(), "talk_decode");
+}
+
+}  // namespace
+
+bool talk_attn_mma_usable(const GqaDims& D, const PagedCache& pc) {
+    const int rep = D.G > 0 ? D.H / D.G : 0;
+    return D.talk && rep >= 1 && rep <= 16 && D.H <= TK_MAX_HEADS && D.G <= TK_UNITS && D.d % 8 == 0 && D.dv % 8 == 0 && D.d <= 128 && D.dv <= 128 && !D.v_is_k && D.softcap == 0.f && !D.rel &&
+           D.dist_exp == 0.f && pc.layer_off % 8 == 0 && pc.page_stride % 8 == 0 && ((long long)pc.page_size * D.d) % 8 == 0 && prompt_keys(D) > 0;
+}
+
+size_t talk_attn_workspace(const GqaDims& D, int n, int splits) { return (size_t)n * splits * talk_part_floats(D) * sizeof(float); }
+
+int launch_talk_attn_mma(const Batch& b, const GqaDims& D, const void* qn, const PagedCache& pc, void* out, float* workspace, int splits, cudaStream_t s) {
+    if (b.n <= 0) return WF_OK;
+    if (!talk_attn_mma_usable(D, pc)) { set_error("attention: the tensor-core form with mixed heads does not take these sizes"); return WF_ERR_UNSUPPORTED; }
+    TalkParams tp{};
+    const int rep = D.H / D.G;
+    if (b.n == b.nseq && workspace && decode_shape(D, tp.kt, tp.nst)) {
+        tp.splits = std::max(1, std::min(splits, 64)); tp.part = workspace;
+        const int mt = (D.H + 15) / 16, it = (D.G * ((D.dv + 15) / 16) + TK_WARPS - 1) / TK_WARPS;
+        int rc;
+        if (mt == 1) rc = it <= 2 ? decode_launch<1, 2>(b, D, qn, pc, tp, s) : it <= 4 ? decode_launch<1, 4>(b, D, qn, pc, tp, s) : it <= 8 ? decode_launch<1, 8>(b, D, qn, pc, tp, s)
+                                                                                                                                             : decode_launch<1, 16>(b, D, qn, pc, tp, s);
+        else rc = it <= 2 ? decode_launch<2, 2>(b, D, qn, pc, tp, s) : it <= 5 ? decode_launch<2, 5>(b, D, qn, pc, tp, s) : decode_launch<2, 8>(b, D, qn, pc, tp, s);
+        if (rc) return rc;
+        const dim3 block((D.dv + 31) / 32 * 32, tp.splits > 4 ? 8 : 4);
+        talk_merge_kernel<<<dim3(b.nseq, D.H), block, ((size_t)tp.splits * D.H + (size_t)block.y * D.dv) * sizeof(float), s>>>(b, D, tp.splits, workspace, (__nv_bfloat16*)out);
+        return launch_check(cudaGetLastError(), "talk_merge");
+    }
+    tp.ub = prompt_units(D);
+    tp.rp2 = 1;
+    while (tp.rp2 < rep) { tp.rp2 <<= 1; ++tp.rp2_log; }
+    tp.tq = tp.ub * 16 / tp.rp2;
+    return prompt_keys(D) == 32 ? prompt_dispatch<32>(b, D, qn, pc, out, tp, s) : prompt_dispatch<16>(b, D, qn, pc, out, tp, s);
 }
 
 }  // namespace seq
