@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """bench.py — decode throughput of the BitNet-2B-4T-shaped hot path on B200.
 
-    python bench.py --gpus N --steps K --warmup W [--impl reference] [--workload bs64|bs1|hybrid|tutizen|nukezen|fivedra]
+    python bench.py --gpus N --steps K --warmup W [--impl reference] [--workload bs64|bs1|hybrid|tutizen|nukezen|fivedra|fuvavik]
 
 --workload hybrid (1 GPU) measures the layer-stack sequence engine (latent attention / gated delta rule / routed feed-forward) instead:
 prefill and decode tok/s at two layer sizes with random weights, per launch-group times, and the BitNet engine at equal size beside it.
@@ -802,8 +802,8 @@ def hybrid_model(cfg, max_tokens, slots, max_step_tokens, shapes=None):
     rng = np.random.default_rng(0)
     base = torch.from_numpy(rng.standard_normal(1 << 22).astype(np.float32)).to(torch.bfloat16).view(torch.int16).numpy().view(np.uint16)
     for name, count, _ in m.engine.expected_tensors():
-        # random values of the scale a trained layer has (~ 1 / sqrt(fan-in)); norm weights near 1
-        if name.endswith(("norm1", "norm2", "norm1b", "norm2b", "final.norm", ".norm")):
+        # random values of the scale a trained layer has (~ 1 / sqrt(fan-in)); norm weights and penalty numbers at 1
+        if name.endswith(("norm1", "norm2", "norm1b", "norm2b", "final.norm", ".norm", ".r1", ".r2")):
             a = np.full(count, 0x3F80, dtype=np.uint16)
         else:
             vals = torch.from_numpy(base.view(np.int16)).view(torch.bfloat16).float().numpy()
@@ -1076,7 +1076,7 @@ FIVEDRA_SIZES = {
 }
 
 
-def fivedra_config(z, f):
+def fivedra_config(z, f, paired_only=False):
     """z: the Nukezen size of the same name (width, heads, window, feed-forward, vocabulary), f: what only this design has"""
     t, g = f["lat"], f["mem"]
     dense = {"kind": "dense", "ff": z["top"] * z["ff"]}
@@ -1089,7 +1089,7 @@ def fivedra_config(z, f):
     par = {"type": "parallel", "mixer": {"left": left, "left_scale": 0.7, "right": right, "right_scale": 0.7}, "mlp": dense}
     layers, shapes = [], {}
     for i in range(z["layers"]):
-        L = (lat, gru, par, par)[i % 4]
+        L = par if paired_only else (lat, gru, par, par)[i % 4]
         layers.append(L)
         if L["type"] == "parallel":
             shapes[f"l{i}.mix.left.rel"] = (z["rel_rows"], z["heads"])
@@ -1135,23 +1135,82 @@ def run_fivedra(args):
     return 0
 
 
+# --workload fuvavik: the Fuvavik design (one layer norm per layer, gated branches; window attention with mixed heads, a logarithmic distance
+# penalty and learned sinks beside gated linear attention; dense gelu units) on the sequence engine at sizes that resemble real layers,
+# random weights, beside the closest existing model on the same engine at equal width / heads / layers / feed-forward size: Fivedra's
+# paired layers (window attention with a distance bias and an extra unit beside a matrix memory with exponential gates).
+FUVAVIK_SIZES = {
+    "w1024": dict(gla=dict(heads=8, d=64, dv=128), rank=64, positions=4096),
+    "w2560": dict(gla=dict(heads=20, d=128, dv=128), rank=128, positions=8192),
+}
+
+
+def fuvavik_config(z, f):
+    """z: the Nukezen size of the same name (width, heads, window, feed-forward, vocabulary), f: what only this design has"""
+    g = f["gla"]
+    left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["d"], "vdim": z["dv"], "scale": z["d"] ** -0.5, "mask": {"size": z["window"]}}
+    right = {"heads": g["heads"], "dim": g["d"], "vdim": g["dv"], "tau": 16.0}
+    L = {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": {"kind": "dense", "ff": z["top"] * z["ff"]}}
+    shapes = {f"l{i}.mix.right.a1": (f["rank"], z["width"]) for i in range(z["layers"])}
+    cfg = {"architecture": "Fuvavik", "vocab": z["vocab"], "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "max_positions": f["positions"],
+           "logit_softcap": 30.0, "layers": [L] * z["layers"]}
+    return cfg, shapes
+
+
+def run_fuvavik(args):
+    from wf_bitnet import _lib
+    torch.cuda.set_device(0)
+    _lib.require_gpu()
+    K, W_ = max(2, args.steps), max(3, args.warmup)
+    peak, peak_src = measured_peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    out, launches = {}, 0
+    for name, f in FUVAVIK_SIZES.items():
+        if args.hybrid_size and name != args.hybrid_size:
+            continue
+        z = NUKEZEN_SIZES[name]
+        prompt = 2048
+        decode_points = [(1, 512), (8, 2048), (64, 4096)] if name == "w2560" else [(1, 512), (8, 1024), (64, 1024)]
+        cfg, shapes = fuvavik_config(z, f)
+        res, n1 = measure_seq_model(cfg, prompt, decode_points, K, shapes)
+        g = f["gla"]
+        # state one decoded token reads and writes per layer (float); cached bytes per layer and 1000 tokens of context
+        res["state_bytes"] = 4 * g["heads"] * g["d"] * g["dv"]
+        res["kv_bytes_per_layer_per_1k_ctx"] = 1000 * z["kv_heads"] * (z["d"] + z["dv"]) * 2
+        fcfg, fshapes = fivedra_config(z, FIVEDRA_SIZES[name], paired_only=True)
+        fres, n2 = measure_seq_model(fcfg, prompt, decode_points, K, fshapes)
+        res["fivedra_paired_equal_size"] = fres
+        launches += n1 + n2
+        out[name] = res
+    clocks = sampler.stop()
+    head = out.get("w2560") or next(iter(out.values()))
+    top = sorted(head["decode"].items())[-1]
+    emit({"metric": "prefill / decode tok/s of the Fuvavik design on the sequence engine beside Fivedra's paired layers at equal size", "workload": "fuvavik",
+          "value": top[1]["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W_, "higher_is_better": True, "dtype": "bf16",
+          "data": "synthetic (random weights; decode contexts are whatever the cache pages hold)", "vs_baseline": None,
+          "config": {"model": "Fuvavik-shaped, " + ", ".join(out), "point": top[0], "l2": "weights per step exceed L2 (126 MB) at w2560; w1024 is L2-resident"},
+          "hbm_peak_gbs": peak, "peak_source": peak_src, "sizes": out, "clocks": clocks, "gpu_launches": launches})
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="bs64", choices=["bs64", "bs1", "hybrid", "tutizen", "nukezen", "fivedra"] + sorted(TP_WORKLOADS))
-    ap.add_argument("--hybrid-size", default="", help="--workload hybrid / tutizen / nukezen / fivedra: run only this size (w1024 | w2560)")
+    ap.add_argument("--workload", default="bs64", choices=["bs64", "bs1", "hybrid", "tutizen", "nukezen", "fivedra", "fuvavik"] + sorted(TP_WORKLOADS))
+    ap.add_argument("--hybrid-size", default="", help="--workload hybrid / tutizen / nukezen / fivedra / fuvavik: run only this size (w1024 | w2560)")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--no-aux", action="store_true", help="skip the batch-1 aux measurement")
     ap.add_argument("--no-tp", action="store_true", help="skip the tensor-parallel suite (aux.tp)")
     args = ap.parse_args()
-    if args.workload in ("hybrid", "tutizen", "nukezen", "fivedra"):
+    if args.workload in ("hybrid", "tutizen", "nukezen", "fivedra", "fuvavik"):
         if args.impl == "reference":
             emit({"impl": "reference", "unavailable": "the reference has no model of this design; its arm is defined for the 2B workloads only"})
             return 0
-        return {"hybrid": run_hybrid, "tutizen": run_tutizen, "nukezen": run_nukezen, "fivedra": run_fivedra}[args.workload](args)
+        return {"hybrid": run_hybrid, "tutizen": run_tutizen, "nukezen": run_nukezen, "fivedra": run_fivedra, "fuvavik": run_fuvavik}[args.workload](args)
     if args.workload in TP_WORKLOADS:
         if args.impl == "reference":
             emit({"impl": "reference", "unavailable": "the reference arm is defined for the 2B workloads (bs64 / bs1) only"})
