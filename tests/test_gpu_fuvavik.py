@@ -168,10 +168,10 @@ def test_feed_forward_and_norm_alone(dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("width,ff", [(40, 28), (40, None), (4200, 16)])
+@pytest.mark.parametrize("width,ff", [(40, 28), (40, None), (38, 28), (1100, 16), (4200, 16), (4201, None), (8300, 16)])
 def test_one_layer_gates_both_branches(dtype, width, ff):
     """The stream after a single layer of a one-layer model: gates, pair norms and the sum in one kernel, with and without a feed-forward,
-    and at a width whose rows exceed the registers of a block.  Opening or closing either gate moves the oracle."""
+    at widths whose rows fit in registers and beyond, aligned and not.  Opening or closing either gate moves the oracle."""
     cfg = config([par(ff=ff)], width=width, vocab=30)
     w = make_weights((cfg, {}), 45)
     toks = tokens_for(cfg, 12, 46)

@@ -25,12 +25,13 @@ constexpr int GA_MAXROT = 256;  // rotated pairs per head
 // One block per token; its warps walk the token's head vectors (H query heads, then G key heads, then G value heads): bias, norm
 // (per head, or over the whole projection with two block-wide sums first), rotation, store.  The cosines and sines of the token's
 // angles are formed once per block in double, so that the float values are the correctly rounded ones at any position.
-template <typename T>
+// MAXD: values a lane holds of one head vector (head sizes up to 32 * MAXD).
+template <typename T, int MAXD>
 __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDims D, const float* __restrict__ proj, int ld, int k_off, int v_off, int g_off,
                                                                    const T* __restrict__ qb, const T* __restrict__ kb, const T* __restrict__ vb, float eps,
                                                                    PagedCache pc, T* __restrict__ qn, float* __restrict__ gate) {
     __shared__ float rot_c[GA_MAXROT], rot_s[GA_MAXROT];
-    __shared__ float vec[GA_WARPS][32 * GA_MAXD];
+    __shared__ float vec[GA_WARPS][32 * MAXD];
     __shared__ float scratch[33];
     const int i = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -81,10 +82,10 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
             src = row + v_off + (size_t)g * D.dv; bias = vb ? vb + (size_t)g * D.dv : nullptr; dim = D.dv; norm = D.v_norm ? 1 : 0; rot = false;
             dst = page + (size_t)D.G * pc.page_size * D.d + ((size_t)g * pc.page_size + slot) * D.dv;
         }
-        float v[GA_MAXD];
+        float v[MAXD];
         float ss = 0.f;
 #pragma unroll
-        for (int t = 0; t < GA_MAXD; ++t) {
+        for (int t = 0; t < MAXD; ++t) {
             const int c = lane + 32 * t;
             v[t] = c < dim ? src[c] + (bias ? to_f(bias[c]) : 0.f) : 0.f;
             ss = fmaf(v[t], v[t], ss);
@@ -93,15 +94,15 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
         if (norm == 1 || norm == 2) { ss = warp_sum(ss); inv = 1.f / sqrtf(ss / (float)dim + eps); }
         else if (norm == 3) inv = inv_all;
 #pragma unroll
-        for (int t = 0; t < GA_MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) v[t] = v[t] * inv * (nw ? to_f(nw[c]) : 1.f); }
+        for (int t = 0; t < MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) v[t] = v[t] * inv * (nw ? to_f(nw[c]) : 1.f); }
         if (rot) {
             float* sv = vec[warp];
             __syncwarp();
 #pragma unroll
-            for (int t = 0; t < GA_MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) sv[c] = v[t]; }
+            for (int t = 0; t < MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) sv[c] = v[t]; }
             __syncwarp();
 #pragma unroll
-            for (int t = 0; t < GA_MAXD; ++t) {
+            for (int t = 0; t < MAXD; ++t) {
                 const int c = lane + 32 * t;
                 if (c < D.rope_dims && c < dim) {
                     int p, other; bool first;
@@ -113,7 +114,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
             }
         }
 #pragma unroll
-        for (int t = 0; t < GA_MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) dst[c] = from_f<T>(v[t]); }
+        for (int t = 0; t < MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) dst[c] = from_f<T>(v[t]); }
     }
     if (gate) {
         const int ng = D.gate_elem ? D.H * D.dv : D.H;
@@ -302,8 +303,11 @@ int launch_gqa_prep(int dt, const Batch& b, const GqaDims& D, const float* proj,
     if (b.n <= 0) return WF_OK;
     if (int rc = check_dims(D)) return rc;
     if (!D.v_is_k && (k_off >= 0) != (v_off >= 0)) { set_error("attention: keys and values are projected together or not at all"); return WF_ERR_INVALID; }
-    if (dt == WF_BF16) gqa_prep_kernel<<<b.n, GA_WARPS * 32, 0, s>>>(b, D, proj, ld, k_off, v_off, g_off, (const __nv_bfloat16*)qb, (const __nv_bfloat16*)kb, (const __nv_bfloat16*)vb, eps, pc, (__nv_bfloat16*)qn, gate);
-    else gqa_prep_kernel<<<b.n, GA_WARPS * 32, 0, s>>>(b, D, proj, ld, k_off, v_off, g_off, (const float*)qb, (const float*)kb, (const float*)vb, eps, pc, (float*)qn, gate);
+    const bool small = D.d <= 128 && D.dv <= 128;
+#define GP_LAUNCH(T, MD) gqa_prep_kernel<T, MD><<<b.n, GA_WARPS * 32, 0, s>>>(b, D, proj, ld, k_off, v_off, g_off, (const T*)qb, (const T*)kb, (const T*)vb, eps, pc, (T*)qn, gate)
+    if (dt == WF_BF16) { if (small) GP_LAUNCH(__nv_bfloat16, 4); else GP_LAUNCH(__nv_bfloat16, GA_MAXD); }
+    else { if (small) GP_LAUNCH(float, 4); else GP_LAUNCH(float, GA_MAXD); }
+#undef GP_LAUNCH
     return launch_check(cudaGetLastError(), "gqa_prep");
 }
 

@@ -22,6 +22,8 @@ namespace {
 constexpr int TK_THREADS = 256, TK_WARPS = 8;
 constexpr int TK_MAX_HEADS = 32, TK_UNITS = 16;      // heads; 16-row units of the prompt form (one per warp)
 
+constexpr int TK_MAX_SPLITS = 32;
+
 struct TalkParams {
     int ub, rp2, rp2_log, tq;    // prompt form: units per key/value head, rows per token (group size rounded up to a power of two), tokens per CTA
     int kt, nst;                 // decode form: keys per tile, staged tiles
@@ -458,23 +460,29 @@ __global__ void __launch_bounds__(TK_THREADS, MT * IT <= 10 ? 2 : 1) talk_decode
             }
         }
         __syncthreads();
-        // ---- online softmax, a warp per head, a lane per key
-        for (int h = warp; h < D.H; h += TK_WARPS) {
-            const int key = t * KT + lane, dist = pos - key;
+        // ---- online softmax, a lane per key, 32 / KT heads per warp at a time
+        const int per = 32 / KT, lk = lane & (KT - 1);
+        for (int h0 = warp * per; h0 < D.H; h0 += TK_WARPS * per) {
+            const int h = h0 + lane / KT, hh = h < D.H ? h : D.H - 1;
+            const int key = t * KT + lk, dist = pos - key;
             float v = -INFINITY;
-            if (lane < KT && dist >= 0 && key >= lo) {
-                const float pen = D.dist_r1 ? D.dist_r1[h] * __log2f(fmaf(D.dist_r2[h], (float)dist, 1.f)) : 0.f;
-                v = fmaf(Sc[h * SS + lane], scale2, -pen);
+            if (dist >= 0 && key >= lo) {
+                const float pen = D.dist_r1 ? D.dist_r1[hh] * __log2f(fmaf(D.dist_r2[hh], (float)dist, 1.f)) : 0.f;
+                v = fmaf(Sc[hh * SS + lk], scale2, -pen);
             }
-            const float mo = hm[h], mn = fmaxf(mo, warp_max(v)), ms = mn == -INFINITY ? 0.f : mn;
-            const float p = exp2f(v - ms), ls = warp_sum(p);
-            if (lane < KT) {
-                const __nv_bfloat16 ph = __float2bfloat16_rn(p);
-                Wh[h * WS + lane] = ph;
-                Wl[h * WS + lane] = __float2bfloat16_rn(p - __bfloat162float(ph));
-            }
+            float mx = v;
+            for (int x = KT / 2; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+            const float mo = hm[hh], mn = fmaxf(mo, mx), ms = mn == -INFINITY ? 0.f : mn;
+            const float p = exp2f(v - ms);
+            float ls = p;
+            for (int x = KT / 2; x > 0; x >>= 1) ls += __shfl_xor_sync(0xffffffffu, ls, x);
             __syncwarp();
-            if (lane == 0) { const float c = exp2f(mo - ms); hc[h] = c; hl[h] = hl[h] * c + ls; hm[h] = mn; }
+            if (h < D.H) {
+                const __nv_bfloat16 ph = __float2bfloat16_rn(p);
+                Wh[h * WS + lk] = ph;
+                Wl[h * WS + lk] = __float2bfloat16_rn(p - __bfloat162float(ph));
+                if (lk == 0) { const float c = exp2f(mo - ms); hc[h] = c; hl[h] = hl[h] * c + ls; hm[h] = mn; }
+            }
         }
         __syncthreads();
         // ---- every head's weights on every key/value head's values
@@ -540,35 +548,50 @@ __global__ void __launch_bounds__(TK_THREADS, MT * IT <= 10 ? 2 : 1) talk_decode
     for (int h = tid; h < D.H; h += TK_THREADS) { ml[h] = hm[h]; ml[D.H + h] = hl[h]; }
 }
 
-// block per (token, head): normalise the source heads over the splits, mix, write.  blockDim = (values rounded up to 32, slices of the sum)
+// block per (token, key/value head, four of its query heads): normalise the source heads over the splits, mix, write; every partial result is
+// read once.  blockDim = (values rounded up to 32, slices of the sum)
+constexpr int TM_HEADS = 4;
 __global__ void talk_merge_kernel(Batch b, GqaDims D, int splits, const float* __restrict__ parts, __nv_bfloat16* __restrict__ out) {
-    extern __shared__ float cf[];                          // [splits][H] factors, then [slices][dv] partial sums
-    const int sq = blockIdx.x, h = blockIdx.y, kv = h / (D.H / D.G), tok = b.seq_start[sq];
-    const int tid = threadIdx.y * blockDim.x + threadIdx.x;
+    extern __shared__ __align__(16) float cf[];            // [splits][H][TM_HEADS] factors, then [slices][TM_HEADS][dv] partial sums
+    const int sq = blockIdx.x, kv = blockIdx.y, rep = D.H / D.G, h0 = kv * rep + blockIdx.z * TM_HEADS, tok = b.seq_start[sq];
+    const int tid = threadIdx.y * blockDim.x + threadIdx.x, cnt = min(TM_HEADS, kv * rep + rep - h0);
     const size_t pf = talk_part_floats(D), mo = (size_t)D.H * D.G * D.dv;
     const float* p = parts + (size_t)sq * splits * pf;
-    float* red = cf + splits * D.H;
+    float* red = cf + splits * D.H * TM_HEADS;
     for (int g = tid; g < D.H; g += blockDim.x * blockDim.y) {
         float m = -INFINITY, l = 0.f;
         for (int s = 0; s < splits; ++s) m = fmaxf(m, p[s * pf + mo + g]);
-        for (int s = 0; s < splits; ++s) { const float f = exp2f(p[s * pf + mo + g] - m); cf[s * D.H + g] = f; l = fmaf(p[s * pf + mo + D.H + g], f, l); }
-        const float w = D.talk[h * D.H + g] * am_inv_sum(D, g, m, l);
-        for (int s = 0; s < splits; ++s) cf[s * D.H + g] *= w;
+        for (int s = 0; s < splits; ++s) l = fmaf(p[s * pf + mo + D.H + g], exp2f(p[s * pf + mo + g] - m), l);
+        const float inv = am_inv_sum(D, g, m, l);
+        float w[TM_HEADS];
+#pragma unroll
+        for (int k = 0; k < TM_HEADS; ++k) w[k] = k < cnt ? D.talk[(h0 + k) * D.H + g] * inv : 0.f;
+        for (int s = 0; s < splits; ++s) {
+            const float f = exp2f(p[s * pf + mo + g] - m);
+            *reinterpret_cast<float4*>(cf + (s * D.H + g) * TM_HEADS) = make_float4(w[0] * f, w[1] * f, w[2] * f, w[3] * f);
+        }
     }
     __syncthreads();
     const int c = threadIdx.x;
-    float v = 0.f;
+    float v[TM_HEADS] = {0.f, 0.f, 0.f, 0.f};
     if (c < D.dv) {
         const float* src = p + (size_t)kv * D.dv + c;
         const int total = splits * D.H;
 #pragma unroll 4
-        for (int e = threadIdx.y; e < total; e += blockDim.y) { const int s = e / D.H, g = e - s * D.H; v = fmaf(cf[e], src[s * pf + (size_t)g * D.G * D.dv], v); }
-        red[threadIdx.y * D.dv + c] = v;
+        for (int e = threadIdx.y; e < total; e += blockDim.y) {
+            const int s = e / D.H, g = e - s * D.H;
+            const float x = src[s * pf + (size_t)g * D.G * D.dv];
+            const float4 f = *reinterpret_cast<const float4*>(cf + e * TM_HEADS);
+            v[0] = fmaf(f.x, x, v[0]); v[1] = fmaf(f.y, x, v[1]); v[2] = fmaf(f.z, x, v[2]); v[3] = fmaf(f.w, x, v[3]);
+        }
+#pragma unroll
+        for (int k = 0; k < TM_HEADS; ++k) red[(threadIdx.y * TM_HEADS + k) * D.dv + c] = v[k];
     }
     __syncthreads();
-    if (threadIdx.y == 0 && c < D.dv) {
-        for (int y = 1; y < (int)blockDim.y; ++y) v += red[y * D.dv + c];
-        out[((size_t)tok * D.H + h) * D.dv + c] = __float2bfloat16_rn(v);
+    for (int e = tid; e < cnt * D.dv; e += blockDim.x * blockDim.y) {
+        float r = 0.f;
+        for (int y = 0; y < (int)blockDim.y; ++y) r += red[y * TM_HEADS * D.dv + e];
+        out[((size_t)tok * D.H + h0) * D.dv + e] = __float2bfloat16_rn(r);
     }
 }
 
@@ -610,7 +633,9 @@ int prompt_dispatch(const Batch& b, const GqaDims& D, const void* qn, const Page
 bool decode_shape(const GqaDims& D, int& kt, int& nst) {
     const int mt = (D.H + 15) / 16, items = D.G * ((D.dv + 15) / 16), it = (items + TK_WARPS - 1) / TK_WARPS;
     if (mt > 2 || it > (mt == 1 ? 16 : 8)) return false;
-    const int shapes[3][2] = {{32, 2}, {16, 2}, {16, 1}};
+    // two blocks per SM hide each other's phases: the larger tile only where two of its blocks fit
+    if (2 * (TalkDecodeShared(D, 32).bytes(D, 2) + 1024) <= 228 * 1024) { kt = 32; nst = 2; return true; }
+    const int shapes[2][2] = {{16, 2}, {16, 1}};
     for (const auto& x : shapes)
         if (TalkDecodeShared(D, x[0]).bytes(D, x[1]) <= TK_SMEM) { kt = x[0]; nst = x[1]; return true; }
     return false;
@@ -641,15 +666,17 @@ int launch_talk_attn_mma(const Batch& b, const GqaDims& D, const void* qn, const
     tp.ps_log = -1;
     for (int k = 0; k < 30; ++k) if (pc.page_size == (1 << k)) tp.ps_log = k;
     if (b.n == b.nseq && workspace && decode_shape(D, tp.kt, tp.nst)) {
-        tp.splits = std::max(1, std::min(splits, 64)); tp.part = workspace;
+        tp.splits = std::max(1, std::min(splits, TK_MAX_SPLITS)); tp.part = workspace;
         const int mt = (D.H + 15) / 16, it = (D.G * ((D.dv + 15) / 16) + TK_WARPS - 1) / TK_WARPS;
         int rc;
         if (mt == 1) rc = it <= 2 ? decode_launch<1, 2>(b, D, qn, pc, tp, s) : it <= 4 ? decode_launch<1, 4>(b, D, qn, pc, tp, s) : it <= 8 ? decode_launch<1, 8>(b, D, qn, pc, tp, s)
                                                                                                                                              : decode_launch<1, 16>(b, D, qn, pc, tp, s);
         else rc = it <= 2 ? decode_launch<2, 2>(b, D, qn, pc, tp, s) : it <= 5 ? decode_launch<2, 5>(b, D, qn, pc, tp, s) : decode_launch<2, 8>(b, D, qn, pc, tp, s);
         if (rc) return rc;
-        const dim3 block((D.dv + 31) / 32 * 32, tp.splits > 4 ? 8 : 4);
-        talk_merge_kernel<<<dim3(b.nseq, D.H), block, ((size_t)tp.splits * D.H + (size_t)block.y * D.dv) * sizeof(float), s>>>(b, D, tp.splits, workspace, (__nv_bfloat16*)out);
+        const int rep = D.H / D.G;
+        const dim3 block((D.dv + 31) / 32 * 32, 8);
+        talk_merge_kernel<<<dim3(b.nseq, D.G, (rep + TM_HEADS - 1) / TM_HEADS), block, ((size_t)tp.splits * D.H + (size_t)block.y * D.dv) * TM_HEADS * sizeof(float), s>>>(
+            b, D, tp.splits, workspace, (__nv_bfloat16*)out);
         return launch_check(cudaGetLastError(), "talk_merge");
     }
     tp.ub = prompt_units(D); tp.rp2 = rows_per_token(D); tp.tq = prompt_tokens(D);

@@ -3,7 +3,7 @@
 // without the correction (u = beta v) is the state-space recurrence S = a S + dt B x^T, y = S^T C with k = B, q = C, v = x, beta = dt, and,
 // with one decay per key row and beta = 1, gated linear attention S = diag(a) S + k v^T.
 // The state is carried per sequence slot across steps.
-#include "seq_kernels.cuh"
+#include "seq_attn_mma.cuh"      // ldmatrix / mma.sync wrappers
 
 namespace wf {
 namespace seq {
@@ -94,20 +94,20 @@ __device__ __forceinline__ void cp_async4(void* smem_dst, const void* gsrc) {
 // DR_PARTS = 4 (32 columns): wider, better coalesced state rows, for single decoded tokens where the state traffic is the cost.
 // VEC: the decay is a vector over the key rows (staged per token like k and q) instead of one number per token.
 // DELTA: the write is corrected by what the state already holds along the key (the delta rule); without it u = beta v.
-template <int DPT, int DR_PARTS, bool VEC, bool DELTA>
+// NC: columns per thread (consecutive ones; 2 halves the shared-memory reads per multiply-add where there are columns and rows enough).
+template <int DPT, int DR_PARTS, bool VEC, bool DELTA, int NC>
 __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDims D, const float* __restrict__ qkv, int ld,
                                                                          const float* __restrict__ beta, const float* __restrict__ decay,
                                                                          float* __restrict__ state, size_t slot_stride, float* __restrict__ o, ScanArgs sa) {
-    constexpr int DR_COLS = DR_THREADS / DR_PARTS;
+    constexpr int DR_COLS = DR_THREADS / DR_PARTS * NC;
     extern __shared__ __align__(16) float sm[];
     // A thread owns DPT consecutive key rows; a token's k / q / decay rows lie in shared memory with 4 floats of padding after every DPT, so
     // that the eight (or four) threads of a column read their parts as 16-byte vectors from distinct banks.
     constexpr int PS = DPT + 4, RS = DR_PARTS * PS;           // floats per part and per token row
     constexpr int tile_floats = (VEC ? 3 : 2) * DR_TT * RS + DR_TT * DR_COLS + 2 * DR_TT;   // k [TT][RS], q [TT][RS], v [TT][cols], beta [TT], decay [TT], vector decay [TT][RS]
     const int sq = sa.pass ? blockIdx.x / sa.nchunks : blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * DR_COLS;
-    const int tid = threadIdx.x, p = tid % DR_PARTS, jl = tid / DR_PARTS, col = col0 + jl;
+    const int tid = threadIdx.x, p = tid % DR_PARTS, jl = tid / DR_PARTS * NC, col = col0 + jl;
     const int dvs = D.dv + D.ones_col;                      // state and output columns: the values, and the all-ones column behind them
-    const bool col_ok = col < dvs;
     const int kh = h / (D.H / D.Hk);
     int start = b.seq_start[sq], len = b.seq_len[sq];
     float* S = state + (size_t)b.seq_slot[sq] * slot_stride + (size_t)h * D.d * dvs;       // where the state is read ...
@@ -127,12 +127,14 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDi
         start += c * sa.chunk;
         len = len - c * sa.chunk < sa.chunk ? len - c * sa.chunk : sa.chunk;
     }
-    float s[DPT];
+    float s[NC][DPT];
 #pragma unroll
-    for (int m = 0; m < DPT; ++m) {
-        const int i = p * DPT + m;
-        s[m] = (S && col_ok && i < D.d) ? S[(size_t)i * dvs + col] : 0.f;
-    }
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int m = 0; m < DPT; ++m) {
+            const int i = p * DPT + m;
+            s[c][m] = (S && col + c < dvs && i < D.d) ? S[(size_t)i * dvs + col + c] : 0.f;
+        }
     const int q_off = (D.q_off >= 0 ? D.q_off : 0) + kh * D.d, k_off = (D.k_off >= 0 ? D.k_off : D.Hk * D.d) + kh * D.d,
               v_off = (D.v_off >= 0 ? D.v_off : 2 * D.Hk * D.d) + h * D.dv;
     auto stage = [&](int buf, int t0) {
@@ -207,65 +209,85 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(Batch b, DeltaDi
                 for (int m4 = 0; m4 < DPT / 4; ++m4) {
                     const float4 gg = gt[m4];
                     const int i = i0 + 4 * m4;
-                    if (i < D.d) s[4 * m4] *= gg.x;
-                    if (i + 1 < D.d) s[4 * m4 + 1] *= gg.y;
-                    if (i + 2 < D.d) s[4 * m4 + 2] *= gg.z;
-                    if (i + 3 < D.d) s[4 * m4 + 3] *= gg.w;
-                }
-            }
-            float rs = 0.f;
-            if (DELTA) {
-                float r[4] = {0.f, 0.f, 0.f, 0.f};            // four chains: the sum over this thread's rows is not one dependent sequence
 #pragma unroll
-                for (int m4 = 0; m4 < DPT / 4; ++m4) {
-                    const float4 kk = kt[m4];
-                    const int i = i0 + 4 * m4;
-                    if (i < D.d) r[0] = fmaf(s[4 * m4], kk.x, r[0]);
-                    if (i + 1 < D.d) r[1] = fmaf(s[4 * m4 + 1], kk.y, r[1]);
-                    if (i + 2 < D.d) r[2] = fmaf(s[4 * m4 + 2], kk.z, r[2]);
-                    if (i + 3 < D.d) r[3] = fmaf(s[4 * m4 + 3], kk.w, r[3]);
+                    for (int c = 0; c < NC; ++c) {
+                        if (i < D.d) s[c][4 * m4] *= gg.x;
+                        if (i + 1 < D.d) s[c][4 * m4 + 1] *= gg.y;
+                        if (i + 2 < D.d) s[c][4 * m4 + 2] *= gg.z;
+                        if (i + 3 < D.d) s[c][4 * m4 + 3] *= gg.w;
+                    }
                 }
-                rs = (r[0] + r[1]) + (r[2] + r[3]);
-                rs += __shfl_xor_sync(0xffffffffu, rs, 1);
-                rs += __shfl_xor_sync(0xffffffffu, rs, 2);
-                if (DR_PARTS == 8) rs += __shfl_xor_sync(0xffffffffu, rs, 4);
             }
-            const float u = bs[t] * (vs[t * DR_COLS + jl] - g * rs);
+            float u[NC];
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                float rs = 0.f;
+                if (DELTA) {
+                    float r[4] = {0.f, 0.f, 0.f, 0.f};        // four chains: the sum over this thread's rows is not one dependent sequence
+#pragma unroll
+                    for (int m4 = 0; m4 < DPT / 4; ++m4) {
+                        const float4 kk = kt[m4];
+                        const int i = i0 + 4 * m4;
+                        if (i < D.d) r[0] = fmaf(s[c][4 * m4], kk.x, r[0]);
+                        if (i + 1 < D.d) r[1] = fmaf(s[c][4 * m4 + 1], kk.y, r[1]);
+                        if (i + 2 < D.d) r[2] = fmaf(s[c][4 * m4 + 2], kk.z, r[2]);
+                        if (i + 3 < D.d) r[3] = fmaf(s[c][4 * m4 + 3], kk.w, r[3]);
+                    }
+                    rs = (r[0] + r[1]) + (r[2] + r[3]);
+                    rs += __shfl_xor_sync(0xffffffffu, rs, 1);
+                    rs += __shfl_xor_sync(0xffffffffu, rs, 2);
+                    if (DR_PARTS == 8) rs += __shfl_xor_sync(0xffffffffu, rs, 4);
+                }
+                u[c] = bs[t] * (vs[t * DR_COLS + jl + c] - g * rs);
+            }
             if (sa.pass == 1) {                               // only the end state is wanted: no read-out
 #pragma unroll
                 for (int m4 = 0; m4 < DPT / 4; ++m4) {
                     const float4 kk = kt[m4];
                     const int i = i0 + 4 * m4;
-                    if (i < D.d) s[4 * m4] = fmaf(kk.x, u, g * s[4 * m4]);
-                    if (i + 1 < D.d) s[4 * m4 + 1] = fmaf(kk.y, u, g * s[4 * m4 + 1]);
-                    if (i + 2 < D.d) s[4 * m4 + 2] = fmaf(kk.z, u, g * s[4 * m4 + 2]);
-                    if (i + 3 < D.d) s[4 * m4 + 3] = fmaf(kk.w, u, g * s[4 * m4 + 3]);
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        if (i < D.d) s[c][4 * m4] = fmaf(kk.x, u[c], g * s[c][4 * m4]);
+                        if (i + 1 < D.d) s[c][4 * m4 + 1] = fmaf(kk.y, u[c], g * s[c][4 * m4 + 1]);
+                        if (i + 2 < D.d) s[c][4 * m4 + 2] = fmaf(kk.z, u[c], g * s[c][4 * m4 + 2]);
+                        if (i + 3 < D.d) s[c][4 * m4 + 3] = fmaf(kk.w, u[c], g * s[c][4 * m4 + 3]);
+                    }
                 }
                 continue;
             }
-            float out[4] = {0.f, 0.f, 0.f, 0.f};
+            float out[NC][4];
+#pragma unroll
+            for (int c = 0; c < NC; ++c) out[c][0] = out[c][1] = out[c][2] = out[c][3] = 0.f;
 #pragma unroll
             for (int m4 = 0; m4 < DPT / 4; ++m4) {
                 const float4 kk = kt[m4], qq = qt[m4];
                 const int i = i0 + 4 * m4;
-                if (i < D.d) { s[4 * m4] = fmaf(kk.x, u, g * s[4 * m4]); out[0] = fmaf(s[4 * m4], qq.x, out[0]); }
-                if (i + 1 < D.d) { s[4 * m4 + 1] = fmaf(kk.y, u, g * s[4 * m4 + 1]); out[1] = fmaf(s[4 * m4 + 1], qq.y, out[1]); }
-                if (i + 2 < D.d) { s[4 * m4 + 2] = fmaf(kk.z, u, g * s[4 * m4 + 2]); out[2] = fmaf(s[4 * m4 + 2], qq.z, out[2]); }
-                if (i + 3 < D.d) { s[4 * m4 + 3] = fmaf(kk.w, u, g * s[4 * m4 + 3]); out[3] = fmaf(s[4 * m4 + 3], qq.w, out[3]); }
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    if (i < D.d) { s[c][4 * m4] = fmaf(kk.x, u[c], g * s[c][4 * m4]); out[c][0] = fmaf(s[c][4 * m4], qq.x, out[c][0]); }
+                    if (i + 1 < D.d) { s[c][4 * m4 + 1] = fmaf(kk.y, u[c], g * s[c][4 * m4 + 1]); out[c][1] = fmaf(s[c][4 * m4 + 1], qq.y, out[c][1]); }
+                    if (i + 2 < D.d) { s[c][4 * m4 + 2] = fmaf(kk.z, u[c], g * s[c][4 * m4 + 2]); out[c][2] = fmaf(s[c][4 * m4 + 2], qq.z, out[c][2]); }
+                    if (i + 3 < D.d) { s[c][4 * m4 + 3] = fmaf(kk.w, u[c], g * s[c][4 * m4 + 3]); out[c][3] = fmaf(s[c][4 * m4 + 3], qq.w, out[c][3]); }
+                }
             }
-            float os = (out[0] + out[1]) + (out[2] + out[3]);
-            os += __shfl_xor_sync(0xffffffffu, os, 1);
-            os += __shfl_xor_sync(0xffffffffu, os, 2);
-            if (DR_PARTS == 8) os += __shfl_xor_sync(0xffffffffu, os, 4);
-            if (p == 0 && col_ok) o[((size_t)(start + t0 + t) * D.H + h) * dvs + col] = os * D.o_scale;
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                float os = (out[c][0] + out[c][1]) + (out[c][2] + out[c][3]);
+                os += __shfl_xor_sync(0xffffffffu, os, 1);
+                os += __shfl_xor_sync(0xffffffffu, os, 2);
+                if (DR_PARTS == 8) os += __shfl_xor_sync(0xffffffffu, os, 4);
+                if (p == 0 && col + c < dvs) o[((size_t)(start + t0 + t) * D.H + h) * dvs + col + c] = os * D.o_scale;
+            }
         }
     }
     if (!S_out) return;
 #pragma unroll
-    for (int m = 0; m < DPT; ++m) {
-        const int i = p * DPT + m;
-        if (col_ok && i < D.d) S_out[(size_t)i * dvs + col] = s[m];
-    }
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int m = 0; m < DPT; ++m) {
+            const int i = p * DPT + m;
+            if (col + c < dvs && i < D.d) S_out[(size_t)i * dvs + col + c] = s[c][m];
+        }
 }
 
 // thread per (sequence, head, state element): chains the chunks' start states from the slot's state and leaves the end state in the slot.
@@ -298,6 +320,82 @@ __global__ void scan_decay_prod_kernel(Batch b, int nd, int chunk, int nchunks, 
     prod[(size_t)(start / chunk + sq + c) * nd + k] = pr;
 }
 
+__device__ __forceinline__ float gla_decay_of(float z, float inv_tau) {        // sigmoid(z)^(1 / tau); ln sigmoid(z) = min(z, 0) - ln(1 + exp(-|z|))
+    return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
+}
+
+// The same on tensor cores (bf16 storage): 64 tokens x 64 channels per block, a warp per 16 tokens.  The float low-rank rows enter as a
+// two-term bf16 split, so that the product sees them to 2^-17; a2 is bf16 as stored.  rp: rank rounded up to 16.
+constexpr int GM_TOK = 64, GM_CH = 64;
+__global__ void __launch_bounds__(128) gla_decay_mma_kernel(int n, int rank, int rp, int nout, const float* __restrict__ a1, int ld, const __nv_bfloat16* __restrict__ a2,
+                                                            const __nv_bfloat16* __restrict__ bias, float inv_tau, float* __restrict__ decay) {
+    extern __shared__ __align__(16) unsigned char gm_raw[];
+    __shared__ float zb[GM_CH];
+    const int S = rp + 8, i0 = blockIdx.x * GM_TOK, c0 = blockIdx.y * GM_CH;
+    __nv_bfloat16* Ah = reinterpret_cast<__nv_bfloat16*>(gm_raw);
+    __nv_bfloat16* Al = Ah + GM_TOK * S;
+    __nv_bfloat16* B = Al + GM_TOK * S;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g4 = lane >> 2, t4 = lane & 3, mi = lane >> 3, rr = lane & 7;
+    if (tid < GM_CH) zb[tid] = c0 + tid < nout ? __bfloat162float(bias[c0 + tid]) : 0.f;
+    for (int e = tid; e < GM_CH * (rp / 8); e += 128) {       // 16 bytes at a time (rank is a multiple of 8)
+        const int c = e / (rp / 8), r = (e - c * (rp / 8)) * 8;
+        const bool ok = c0 + c < nout && r < rank;
+        am_cp16(smem_u32(B + c * S + r), ok ? a2 + (size_t)(c0 + c) * rank + r : a2, ok);
+    }
+    am_commit();
+    for (int r = lane; r < rp; r += 32) {
+        float v[GM_TOK / 4];                                  // independent loads: all in flight at once
+#pragma unroll
+        for (int k = 0; k < GM_TOK / 4; ++k) { const int t = i0 + warp + 4 * k; v[k] = t < n && r < rank ? a1[(size_t)t * ld + r] : 0.f; }
+#pragma unroll
+        for (int k = 0; k < GM_TOK / 4; ++k) {
+            const int at = (warp + 4 * k) * S + r;
+            const __nv_bfloat16 hi = __float2bfloat16_rn(v[k]);
+            Ah[at] = hi;
+            Al[at] = __float2bfloat16_rn(v[k] - __bfloat162float(hi));
+        }
+    }
+    am_wait<0>();
+    __syncthreads();
+    if (i0 + warp * 16 >= n) return;
+    float acc[GM_CH / 8][4];
+#pragma unroll
+    for (int j = 0; j < GM_CH / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    const uint32_t ah = smem_u32(Ah), al = smem_u32(Al), bb = smem_u32(B);
+    for (int k = 0; k < rp; k += 16) {
+        uint32_t fh[4], fl[4];
+        const uint32_t at = (uint32_t)((warp * 16 + (lane & 15)) * S + k + (lane >> 4) * 8) * 2u;
+        am_ldsm_x4(fh, ah + at);
+        am_ldsm_x4(fl, al + at);
+#pragma unroll
+        for (int jp = 0; jp < GM_CH / 16; ++jp) {
+            uint32_t f[4];
+            am_ldsm_x4(f, bb + (uint32_t)((jp * 16 + (mi >> 1) * 8 + rr) * S + k + (mi & 1) * 8) * 2u);
+            am_mma(acc[2 * jp], fh, f[0], f[1]);
+            am_mma(acc[2 * jp + 1], fh, f[2], f[3]);
+            am_mma(acc[2 * jp], fl, f[0], f[1]);
+            am_mma(acc[2 * jp + 1], fl, f[2], f[3]);
+        }
+    }
+    // every value is finished before the first is stored: the special functions of independent values overlap
+#pragma unroll
+    for (int j = 0; j < GM_CH / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[j][e] = gla_decay_of(acc[j][e] + zb[j * 8 + 2 * t4 + (e & 1)], inv_tau);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int i = i0 + warp * 16 + g4 + 8 * k;
+        if (i >= n) continue;
+        float* row = decay + (size_t)i * nout + c0 + 2 * t4;
+#pragma unroll
+        for (int j = 0; j < GM_CH / 8; ++j) {
+            const int c = c0 + j * 8 + 2 * t4;
+            if ((nout & 1) == 0 && c < nout) *reinterpret_cast<float2*>(row + j * 8) = make_float2(acc[j][2 * k], acc[j][2 * k + 1]);
+            else { if (c < nout) row[j * 8] = acc[j][2 * k]; if (c + 1 < nout) row[j * 8 + 1] = acc[j][2 * k + 1]; }
+        }
+    }
+}
+
 // decay of gated linear attention: a thread owns one output channel and GD_TOK tokens; the tokens' low-rank rows lie in shared memory
 constexpr int GD_TOK = 8, GD_THREADS = 128;
 template <typename T>
@@ -324,10 +422,7 @@ __global__ void __launch_bounds__(GD_THREADS) gla_decay_kernel(int n, int rank, 
     }
 #pragma unroll
     for (int t = 0; t < GD_TOK; ++t)
-        if (i0 + t < n) {
-            const float z = acc[t];                  // ln sigmoid(z) = min(z, 0) - ln(1 + exp(-|z|))
-            decay[(size_t)(i0 + t) * nout + c] = expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau);
-        }
+        if (i0 + t < n) decay[(size_t)(i0 + t) * nout + c] = gla_decay_of(acc[t], inv_tau);
 }
 
 template <typename T>
@@ -364,25 +459,32 @@ template <bool VEC, bool DELTA>
 int delta_rule_launch(const Batch& b, const DeltaDims& D, const float* qkv, int ld, const float* beta, const float* decay, float* state,
                       size_t slot_stride, float* o, cudaStream_t s, ScanArgs sa = ScanArgs()) {
     const bool decode = b.n == b.nseq;                     // every sequence brings one token
-    const int parts = decode ? 4 : 8, cols = DR_THREADS / parts;
+    // two columns per thread where a block's 32 columns exist and the chunks in parallel still fill the machine
+    const bool wide = !DELTA && sa.pass && D.d <= 128 && D.dv + D.ones_col >= 32 && (long long)b.nseq * sa.nchunks * D.H * ((D.dv + D.ones_col + 31) / 32) >= 4 * sm_count();
+    const int parts = decode ? 4 : 8, cols = DR_THREADS / parts * (wide ? 2 : 1);
     dim3 grid(sa.pass ? b.nseq * sa.nchunks : b.nseq, D.H, (D.dv + D.ones_col + cols - 1) / cols);
     const int dpt_raw = (D.d + parts - 1) / parts, dpt_t = dpt_raw <= 8 ? 8 : (dpt_raw <= 16 ? 16 : (dpt_raw <= 32 ? 32 : 64));
     const size_t smem = 2 * ((size_t)(VEC ? 3 : 2) * DR_TT * parts * (dpt_t + 4) + DR_TT * cols + 2 * DR_TT) * sizeof(float);   // two token groups, padded rows
     static DevOnce once;
     if (once.need()) {
-#define DR_ATTR(dp, pa) cudaFuncSetAttribute(delta_rule_kernel<dp, pa, VEC, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
+#define DR_ATTR(dp, pa) cudaFuncSetAttribute(delta_rule_kernel<dp, pa, VEC, DELTA, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
         DR_ATTR(8, 8); DR_ATTR(16, 8); DR_ATTR(32, 8); DR_ATTR(64, 8); DR_ATTR(8, 4); DR_ATTR(16, 4); DR_ATTR(32, 4); DR_ATTR(64, 4);
 #undef DR_ATTR
+        if (!DELTA) {
+            cudaFuncSetAttribute(delta_rule_kernel<8, 8, VEC, DELTA, DELTA ? 1 : 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+            cudaFuncSetAttribute(delta_rule_kernel<16, 8, VEC, DELTA, DELTA ? 1 : 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+        }
     }
     const int dpt = (D.d + parts - 1) / parts;
     {   // 16-byte staging copies when every row the kernel stages starts aligned and has a multiple of 4 entries
         const int qo = D.q_off >= 0 ? D.q_off : 0, ko = D.k_off >= 0 ? D.k_off : D.Hk * D.d, vo = D.v_off >= 0 ? D.v_off : 2 * D.Hk * D.d;
         sa.v4 = D.d % 4 == 0 && D.dv % 4 == 0 && ld % 4 == 0 && qo % 4 == 0 && ko % 4 == 0 && vo % 4 == 0 && ((uintptr_t)qkv & 15) == 0 && ((uintptr_t)decay & 15) == 0;
     }
-#define DR_LAUNCH(dp, pa) delta_rule_kernel<dp, pa, VEC, DELTA><<<grid, DR_THREADS, smem, s>>>(b, D, qkv, ld, beta, decay, state, slot_stride, o, sa)
+#define DR_LAUNCH(dp, pa, nc) delta_rule_kernel<dp, pa, VEC, DELTA, nc><<<grid, DR_THREADS, smem, s>>>(b, D, qkv, ld, beta, decay, state, slot_stride, o, sa)
     if (D.d > 256 || smem > 160 * 1024) { set_error("delta: key dimension %d above the supported 256", D.d); return WF_ERR_UNSUPPORTED; }
-    if (decode) { if (dpt <= 8) DR_LAUNCH(8, 4); else if (dpt <= 16) DR_LAUNCH(16, 4); else if (dpt <= 32) DR_LAUNCH(32, 4); else DR_LAUNCH(64, 4); }
-    else { if (dpt <= 8) DR_LAUNCH(8, 8); else if (dpt <= 16) DR_LAUNCH(16, 8); else if (dpt <= 32) DR_LAUNCH(32, 8); else DR_LAUNCH(64, 8); }
+    if (wide) { if (dpt <= 8) DR_LAUNCH(8, 8, (DELTA ? 1 : 2)); else DR_LAUNCH(16, 8, (DELTA ? 1 : 2)); }
+    else if (decode) { if (dpt <= 8) DR_LAUNCH(8, 4, 1); else if (dpt <= 16) DR_LAUNCH(16, 4, 1); else if (dpt <= 32) DR_LAUNCH(32, 4, 1); else DR_LAUNCH(64, 4, 1); }
+    else { if (dpt <= 8) DR_LAUNCH(8, 8, 1); else if (dpt <= 16) DR_LAUNCH(16, 8, 1); else if (dpt <= 32) DR_LAUNCH(32, 8, 1); else DR_LAUNCH(64, 8, 1); }
 #undef DR_LAUNCH
     return launch_check(cudaGetLastError(), "delta_rule");
 }
@@ -432,6 +534,15 @@ int launch_delta_post(int dt, const DeltaDims& D, int n, const float* o, const v
 
 int launch_gla_decay(int dt, int n, int rank, int nout, const float* a1, int ld, const void* a2, const void* bias, float tau, float* decay, cudaStream_t s) {
     if (n <= 0) return WF_OK;
+    const int rp = (rank + 15) / 16 * 16;
+    const size_t mma_smem = (size_t)(2 * GM_TOK + GM_CH) * (rp + 8) * 2;
+    if (dt == WF_BF16 && rank > 0 && tau > 0.f && rank % 8 == 0 && mma_smem <= 160 * 1024) {
+        static DevOnce once;
+        if (once.need()) cudaFuncSetAttribute(gla_decay_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+        gla_decay_mma_kernel<<<dim3((n + GM_TOK - 1) / GM_TOK, (nout + GM_CH - 1) / GM_CH), 128, mma_smem, s>>>(n, rank, rp, nout, a1, ld, (const __nv_bfloat16*)a2,
+                                                                                                              (const __nv_bfloat16*)bias, 1.f / tau, decay);
+        return launch_check(cudaGetLastError(), "gla_decay_mma");
+    }
     const size_t smem = (size_t)rank * GD_TOK * sizeof(float);
     if (rank <= 0 || !(tau > 0.f) || smem > 48 * 1024) { set_error("gla: decay projection of rank %d, tau %g", rank, tau); return WF_ERR_UNSUPPORTED; }
     const dim3 grid((n + GD_TOK - 1) / GD_TOK, (nout + GD_THREADS - 1) / GD_THREADS);

@@ -502,10 +502,10 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     if (e->dt == WF_BF16 && e->attn_mma >= 1 && D.talk && !gate && talk_attn_mma_usable(D, pc)) {
         int splits = 1;
         if (n == b.nseq) {
-            splits = (2 * sm_count() + n - 1) / n;           // one block per token and split runs every head; one is resident per SM
+            // one block per token and split runs every head, two are resident per SM: one wave of them, at most sixteen splits to merge
+            splits = std::min(2 * sm_count() / n, 16);
             if (splits > span / 128) splits = (int)(span / 128);
             while (splits > 1 && talk_attn_workspace(D, n, splits) > e->gqa_ws_bytes) --splits;
-            if (splits > 64) splits = 64;
             if (splits < 1) splits = 1;
         }
         if ((rc = launch_talk_attn_mma(b, D, e->qn, pc, e->og, e->gqa_ws, splits, s))) return rc;

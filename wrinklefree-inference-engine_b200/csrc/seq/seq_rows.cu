@@ -333,10 +333,105 @@ __global__ void __launch_bounds__(512) branch_add_norm_kernel(float* __restrict_
         h[base + c] = from_f<T>((row[c] - mean) * inv * (w_offset + to_f(w[c])) + (b ? to_f(b[c]) : 0.f));
 }
 
+template <typename T> __device__ __forceinline__ float4 load4(const T* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&v)[4]) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+// The same with four consecutive elements per load, every input of a row requested before the first is used; a thread owns NV groups of four,
+// blockDim.x * NV * 4 >= W.
+template <typename T, int NV>
+__global__ void __launch_bounds__(1024) branch_add_norm_vec_kernel(float* __restrict__ x, BranchSum bs, const T* __restrict__ w, const T* __restrict__ b, float w_offset, float eps,
+                                                                   int W, T* __restrict__ h) {
+    __shared__ float scratch[33];
+    const size_t base = (size_t)blockIdx.x * W;
+    const float* gate = bs.gate ? bs.gate + (size_t)blockIdx.x * bs.ldg : nullptr;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 xv[NV], v1[NV], v2[NV], v3[NV], g1[NV], g2[NV];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * 4;
+        const bool in = c < W;
+        xv[k] = in ? load4(x + base + c) : zero;
+        v1[k] = in && bs.y1 ? load4(bs.y1 + base + c) : zero;
+        v2[k] = in && bs.y2 ? load4(bs.y2 + base + c) : zero;
+        v3[k] = in && bs.y3 ? load4(bs.y3 + base + c) : zero;
+        g1[k] = in && gate ? load4(gate + c) : zero;
+        g2[k] = in && gate && bs.y3 ? load4(gate + W + c) : zero;
+    }
+    float f1 = bs.a1, f2 = bs.a2;
+    if (bs.pw1 && bs.y1) {
+        float s1 = 0.f, s2 = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            s1 += v1[k].x * v1[k].x + v1[k].y * v1[k].y + v1[k].z * v1[k].z + v1[k].w * v1[k].w;
+            s2 += v2[k].x * v2[k].x + v2[k].y * v2[k].y + v2[k].z * v2[k].z + v2[k].w * v2[k].w;
+        }
+        f1 *= 1.f / sqrtf(block_sum(s1, scratch) / (float)W + eps);
+        if (bs.y2) f2 *= 1.f / sqrtf(block_sum(s2, scratch) / (float)W + eps);
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * 4;
+        if (c >= W || !bs.y1) { sum += xv[k].x + xv[k].y + xv[k].z + xv[k].w; continue; }
+        const float4 one = make_float4(1.f, 1.f, 1.f, 1.f);
+        const float4 p1 = bs.pw1 ? load4((const T*)bs.pw1 + c) : one, p2 = bs.pw2 && bs.y2 ? load4((const T*)bs.pw2 + c) : one;
+        const float4 b1 = gate ? load4((const T*)bs.gb1 + c) : zero, b2 = gate && bs.y3 ? load4((const T*)bs.gb2 + c) : zero;
+        const float a[4] = {v1[k].x * p1.x, v1[k].y * p1.y, v1[k].z * p1.z, v1[k].w * p1.w}, d[4] = {v2[k].x * p2.x, v2[k].y * p2.y, v2[k].z * p2.z, v2[k].w * p2.w};
+        const float u[4] = {v3[k].x, v3[k].y, v3[k].z, v3[k].w}, o[4] = {xv[k].x, xv[k].y, xv[k].z, xv[k].w};
+        const float z1[4] = {g1[k].x + b1.x, g1[k].y + b1.y, g1[k].z + b1.z, g1[k].w + b1.w}, z2[4] = {g2[k].x + b2.x, g2[k].y + b2.y, g2[k].z + b2.z, g2[k].w + b2.w};
+        float r[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float m = f1 * a[e] + f2 * d[e];
+            r[e] = o[e] + (gate ? sigmoid_f(z1[e]) * m + sigmoid_f(z2[e]) * u[e] : m + u[e]);
+            sum += r[e];
+        }
+        store4(x + base + c, r);
+        xv[k] = make_float4(r[0], r[1], r[2], r[3]);
+    }
+    if (!w) return;
+    const float mean = b ? block_sum(sum, scratch) / (float)W : 0.f;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        if ((threadIdx.x + k * blockDim.x) * 4 >= W) continue;
+        xv[k].x -= mean; xv[k].y -= mean; xv[k].z -= mean; xv[k].w -= mean;
+        ss += xv[k].x * xv[k].x + xv[k].y * xv[k].y + xv[k].z * xv[k].z + xv[k].w * xv[k].w;
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, scratch) / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * 4;
+        if (c >= W) continue;
+        const float4 wv = load4(w + c), bv = b ? load4(b + c) : zero;
+        const float r[4] = {xv[k].x * inv * (w_offset + wv.x) + bv.x, xv[k].y * inv * (w_offset + wv.y) + bv.y, xv[k].z * inv * (w_offset + wv.z) + bv.z,
+                            xv[k].w * inv * (w_offset + wv.w) + bv.w};
+        store4(h + base + c, r);
+    }
+}
+
 int launch_branch_add_norm(int dt, float* x, const BranchSum& bs, const void* w, const void* b, float w_offset, float eps, int n, int W, void* h, cudaStream_t s) {
     if (n <= 0) return WF_OK;
     if ((bs.y2 || bs.y3) && !bs.y1) { set_error("branch_add_norm: a second output without a first"); return WF_ERR_INVALID; }
     if (bs.y2 && (bs.pw1 != nullptr) != (bs.pw2 != nullptr)) { set_error("branch_add_norm: both outputs of a pair are normed or none"); return WF_ERR_INVALID; }
+    // rows of up to 8192 elements that start 16-byte aligned stay in registers, four elements per load
+    if (W % 4 == 0 && W <= 8192 && bs.ldg % 4 == 0 && ((uintptr_t)bs.gate & 15) == 0) {
+        const int nv = W <= 1024 ? 1 : 2, threads = (W / 4 + nv * 32 - 1) / (nv * 32) * 32;
+#define BA_LAUNCH(T, NV) branch_add_norm_vec_kernel<T, NV><<<n, threads, 0, s>>>(x, bs, (const T*)w, (const T*)b, w_offset, eps, W, (T*)h)
+        if (dt == WF_BF16) { if (nv == 1) BA_LAUNCH(__nv_bfloat16, 1); else BA_LAUNCH(__nv_bfloat16, 2); }
+        else { if (nv == 1) BA_LAUNCH(float, 1); else BA_LAUNCH(float, 2); }
+#undef BA_LAUNCH
+        return launch_check(cudaGetLastError(), "branch_add_norm_vec");
+    }
     if (dt == WF_BF16) branch_add_norm_kernel<<<n, row_threads(W), 0, s>>>(x, bs, (const __nv_bfloat16*)w, (const __nv_bfloat16*)b, w_offset, eps, W, (__nv_bfloat16*)h);
     else branch_add_norm_kernel<<<n, row_threads(W), 0, s>>>(x, bs, (const float*)w, (const float*)b, w_offset, eps, W, (float*)h);
     return launch_check(cudaGetLastError(), "branch_add_norm");
