@@ -22,7 +22,8 @@ extern "C" {
 #define WF_SEQ_GLA 6               /* gated linear attention: matrix state per head, one decay per key channel, no write correction */
 
 /* how a layer wraps its sublayers */
-#define WF_SEQ_BLOCK_SANDWICH 0    /* x += norm_b(sub(conv(norm_a(x)))): grouped norms before and after, input convolution with carried tail */
+#define WF_SEQ_BLOCK_SANDWICH 0    /* x += norm_b(sub(conv(norm_a(x)))): norms before and after; grouped RMS norms with an input convolution
+                                    * and its carried tail, or (norm_kind) element-wise norms without one */
 #define WF_SEQ_BLOCK_POST 1        /* x += residual_mult * gain * rms(sub(x)): the sublayer reads the stream, ONE gain per norm */
 #define WF_SEQ_BLOCK_PARALLEL 2    /* x += mixer(norm1(x)) + ff(norm2(x)): both branches read the same stream, each behind its own weighted norm
                                     * (one norm for both with one_norm; either branch times a sigmoid gate with branch_gates) */
@@ -34,7 +35,12 @@ extern "C" {
 #define WF_SEQ_ACT_SILU 0          /* silu(g) * u */
 #define WF_SEQ_ACT_CLAMPED 1       /* g = min(g, limit), u = clamp(u, -limit, limit); g * sigmoid(1.702 g) * (u + 1) */
 #define WF_SEQ_ACT_GELU_TANH 2     /* gelu(g) * u, gelu in its tanh form */
-#define WF_SEQ_ACT_RELU2 3         /* relu(u)^2, no gate: the dense feed-forward has 'mlp.up' and 'mlp.down' only */
+#define WF_SEQ_ACT_RELU2 3         /* relu(u)^2, no gate: the feed-forward (or expert) has 'up' and 'down' only */
+#define WF_SEQ_ACT_GELU_ERF 4      /* u (1 + erf(u / sqrt 2)) / 2, no gate either */
+
+/* wf_seq_config.norm_kind */
+#define WF_SEQ_NORM_RMS 0
+#define WF_SEQ_NORM_DYN_TANH 1     /* tanh(alpha x) w + b per element, no statistics: tensors '<norm>', '<norm>.b' [width], '<norm>.alpha' [1] */
 
 /* wf_seq_layer.qk_norm of grouped-query attention */
 #define WF_SEQ_QKNORM_NONE 0
@@ -105,7 +111,8 @@ typedef struct wf_seq_layer {
      * and cosines and sines are multiplied by 0.1 ln(rope_factor) + 1.  (The engine tabulates the frequencies once, in double.) */
     float rope_factor, rope_orig, rope_fast, rope_slow;
     /* grouped-query attention: v_is_k = 1: there is no value projection; the values are the keys as cached (vdim == dim), and a page
-     * holds the keys only. */
+     * holds the keys only.  v_is_k = 2: no value projection either, but the values are the keys as projected, before norm and rotation;
+     * a page holds both. */
     int v_is_k;
     /* WF_SEQ_MINGRU: `vdim` channels (heads = dim = 1).  z = sigmoid(W_z x + b_z), u = W_x x + b_x, c = u + 1/2 (u >= 0) or sigmoid(u);
      * S <- (1 - z) S + z c per channel; output W_o (S * silu(W_g x)).  Tensors mix.z, mix.z.b, mix.x, mix.x.b, mix.g, mix.o.
@@ -128,6 +135,12 @@ typedef struct wf_seq_layer {
      * its root mean square, times mix.norm [vdim], times silu(W_g x), then W_o.  Tensors mix.q, mix.k, mix.v, mix.g, mix.a1, mix.a2, mix.a2.b,
      * mix.norm, mix.o. */
     float decay_tau;
+    /* grouped-query attention, further.  keep_first > 0: positions below it stay visible to every later one however far the window has
+     * moved on (not with chunk or talk).  rope_factor as for latent attention. */
+    int keep_first;
+    /* routed feed-forward, further.  no_correction = 1: the choice is made from the scores alone (no tensor mlp.correction).  shared_plain =
+     * 1: the shared expert's output is added as it is (no tensor mlp.shared.sg). */
+    int no_correction, shared_plain;
 } wf_seq_layer;
 
 typedef struct wf_seq_config {
@@ -154,6 +167,13 @@ typedef struct wf_seq_config {
                                     * 'l<i>.rg1.b' for the mixer, 'l<i>.rg2', 'l<i>.rg2.b' for the feed-forward) */
     int max_positions;             /* pos_embed = 2: rows of the position table; no sequence grows longer */
     float logit_softcap;           /* > 0: logits <- cap * tanh(logits / cap) */
+    int norm_kind;                 /* WF_SEQ_NORM_*: of every layer norm and the final norm.  WF_SEQ_NORM_DYN_TANH: WF_SEQ_BLOCK_SANDWICH with
+                                    * canon_taps = 0 (no input convolution) */
+    /* loop_times > 1: layers loop_start .. loop_stop - 1 run that many times in a row with the same tensors, every pass with cache and state of
+     * its own, then the rest follow; right before every pass but the first the embedding row is added to the stream (WF_SEQ_NORM_DYN_TANH form
+     * only, without position embeddings).  `n_layers` counts layers; what runs is wf_seq_layer_runs() of them, and the layer index of
+     * wf_seq_run_part and of the layer tap counts runs. */
+    int loop_start, loop_stop, loop_times;
 } wf_seq_config;
 
 typedef struct wf_seq_engine wf_seq_engine;
@@ -162,6 +182,7 @@ int wf_seq_available(void);
 int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layers, wf_seq_engine** out);
 void wf_seq_destroy(wf_seq_engine* e);
 size_t wf_seq_device_bytes(const wf_seq_engine* e);
+int wf_seq_layer_runs(const wf_seq_engine* e);
 /* Upload one checkpoint tensor by its checkpoint name ('embed', 'l3.mix.q', 'l0.mlp.e7.down', ...); data holds `count` elements of the
  * engine's dtype (host or device memory).  The engine lays the pieces out for its kernels (fused projections, stacked experts). */
 int wf_seq_set_tensor(wf_seq_engine* e, const char* name, const void* data, size_t count, int is_host);
@@ -190,11 +211,11 @@ void* wf_seq_logits_device(wf_seq_engine* e);
 int wf_seq_launches_last_step(const wf_seq_engine* e);
 
 /* Parity taps.  layer_tap: when not null, the residual stream after every layer of the next steps is copied there
- * (float [n_layers, n, width], n = tokens of the step).  wf_seq_run_part runs ONE part of one layer on given float rows (host memory,
+ * (float [layer runs, n, width], n = tokens of the step).  wf_seq_run_part runs ONE part of one layer on given float rows (host memory,
  * [n, width]) through the same kernels, caches and state as wf_seq_step, and returns that part's float output [n, width]:
  * 0 first norm, 1 input convolution of the mixer (carried state), 2 the mixer, 3 the feed-forward, 4 input convolution of the
- * feed-forward (1 and 4: WF_SEQ_BLOCK_SANDWICH only; part 0 of WF_SEQ_BLOCK_POST is residual_mult * gain * rms(rows)), 5 second norm
- * (WF_SEQ_BLOCK_PARALLEL with two norms only).
+ * feed-forward (1 and 4: input convolutions only; part 0 of WF_SEQ_BLOCK_POST is residual_mult * gain * rms(rows)), 5 second norm
+ * (WF_SEQ_BLOCK_PARALLEL with two norms, WF_SEQ_NORM_DYN_TANH), 6 and 7 the norms behind the mixer and the feed-forward (WF_SEQ_NORM_DYN_TANH).
  * Sequence lengths advance as in a step. */
 int wf_seq_set_layer_tap(wf_seq_engine* e, float* host);
 int wf_seq_run_part(wf_seq_engine* e, int layer, int part, int nseq, const int32_t* slots, const int32_t* counts, const float* in_host,

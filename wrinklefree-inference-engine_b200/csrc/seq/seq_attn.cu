@@ -1,7 +1,7 @@
 // Grouped-query softmax attention over a paged cache of per-head keys and values.  Positions can enter through a rotation of queries and
 // keys (partial, pairs interleaved or split in halves), through a linear distance penalty per head (score -= slope_h * (i - j),
 // slope_h = 2^(-dist_exp (h + 1) / H)) or through a learned bias by distance; the visible keys are the causal ones inside a sliding window
-// and / or inside the query's own chunk of positions; scores can be capped by a tanh, lowered by a logarithm of the distance, and the softmax
+// (beside a few first positions that stay visible) and / or inside the query's own chunk of positions; scores can be capped by a tanh, lowered by a logarithm of the distance, and the softmax
 // denominator can carry an extra one or a learned sink per head; the heads' weights can be mixed by a matrix before they meet the values.
 // Queries, keys and values can be normalised before use (per head, with or without weights, or over the whole projection; the cache holds
 // keys and values in that form), and the output can be multiplied by a sigmoid gate computed from the layer input, per head or per element.
@@ -48,8 +48,8 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
     if (half > 0) {
         const double lb = log2((double)D.rope_base);
         for (int p = threadIdx.x; p < half; p += blockDim.x) {
-            const double a = (double)pos * exp2(-2.0 * (double)p / (double)D.rope_dims * lb);
-            rot_c[p] = (float)cos(a); rot_s[p] = (float)sin(a);
+            const double a = (double)pos * (D.freq ? D.freq[p] : exp2(-2.0 * (double)p / (double)D.rope_dims * lb));
+            rot_c[p] = (float)cos(a) * D.mscale; rot_s[p] = (float)sin(a) * D.mscale;
         }
     }
     float inv_q = 1.f, inv_k = 1.f;
@@ -122,8 +122,8 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
     }
 }
 
-// One block per (token, head).  Its warps take the visible keys round-robin, a warp one key at a time with its lanes over the dimensions;
-// running max / sum / weighted value sum per warp, merged through shared memory.
+// One block per (token, head).  Its warps take the visible keys (the kept first ones, then the window) round-robin, a warp one key at a time
+// with its lanes over the dimensions; running max / sum / weighted value sum per warp, merged through shared memory.
 template <typename T>
 __global__ void __launch_bounds__(GA_WARPS * 32) gqa_attn_kernel(Batch b, GqaDims D, const T* __restrict__ qn, const float* __restrict__ gate, PagedCache pc,
                                                                    T* __restrict__ out) {
@@ -134,6 +134,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_attn_kernel(Batch b, GqaDim
     const int g = h / (D.H / D.G);
     int lo = pos - D.window + 1 > 0 ? pos - D.window + 1 : 0;
     if (D.chunk > 0) { const int c0 = pos / D.chunk * D.chunk; if (c0 > lo) lo = c0; }
+    const int kept = D.keep_first < lo ? D.keep_first : lo;          // first positions that the window itself does not reach
     const int32_t* bt = pc.block_table + (size_t)b.seq_slot[sq] * pc.max_blocks;
     const float slope = D.dist_exp > 0.f ? exp2f(-D.dist_exp * (float)(h + 1) / (float)D.H) : 0.f;
     const T* qh = qn + ((size_t)i * D.H + h) * D.d;
@@ -142,7 +143,8 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_attn_kernel(Batch b, GqaDim
 #pragma unroll
     for (int t = 0; t < GA_MAXD; ++t) { const int c = lane + 32 * t; qreg[t] = c < D.d ? to_f(qh[c]) : 0.f; acc[t] = 0.f; }
     float m = -INFINITY, l = 0.f;
-    for (int j = lo + warp; j <= pos; j += GA_WARPS) {
+    for (int u = warp; u < kept + pos - lo + 1; u += GA_WARPS) {
+        const int j = u < kept ? u : lo + u - kept;
         const T* page = (const T*)pc.pool + (size_t)bt[j / pc.page_size] * pc.page_stride + pc.layer_off;
         const int slot = j % pc.page_size;
         const T* kr = page + k_base + (size_t)slot * D.d;
@@ -290,6 +292,7 @@ int check_dims(const GqaDims& D) {
     if (D.rope_dims < 0 || (D.rope_dims & 1) || D.rope_dims > D.d || D.rope_dims / 2 > GA_MAXROT) { set_error("attention: %d rotated entries of %d", D.rope_dims, D.d); return WF_ERR_INVALID; }
     if (D.qk_norm >= 2 && (!D.q_norm_w || !D.k_norm_w)) { set_error("attention: the query / key norm has no weights"); return WF_ERR_INVALID; }
     if (D.v_is_k && D.dv != D.d) { set_error("attention: values that are the keys have the keys' size (%d / %d)", D.d, D.dv); return WF_ERR_INVALID; }
+    if (D.keep_first < 0 || (D.keep_first > 0 && (D.chunk > 0 || D.talk))) { set_error("attention: %d kept first positions (not with chunks or mixed heads)", D.keep_first); return WF_ERR_UNSUPPORTED; }
     if (D.chunk < 0 || (D.rel && D.rel_n < 1)) { set_error("attention: chunk %d, %d bias rows", D.chunk, D.rel_n); return WF_ERR_INVALID; }
     return WF_OK;
 }

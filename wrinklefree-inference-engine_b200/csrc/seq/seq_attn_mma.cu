@@ -109,12 +109,17 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
     // key range of the tile: every key some row of the tile may see, cut into AM_KT-key tiles aligned to multiples of AM_KT
     int lo_all = pos0 - D.window + 1 > 0 ? pos0 - D.window + 1 : 0;
     if (D.chunk > 0) { const int c0 = pos0 / D.chunk * D.chunk; if (c0 > lo_all) lo_all = c0; }
-    int t_lo = lo_all / AM_KT, t_hi = pos_last / AM_KT;    // inclusive
+    // The tiles to walk are numbered u_lo .. u_hi: first those of the kept first positions that lie before the window's first tile, then the
+    // window's, t_lo .. the tile of the last position.
+    const int t_lo = lo_all / AM_KT;
+    const int kept_t = min((D.keep_first + AM_KT - 1) / AM_KT, t_lo);
+    int u_lo = 0, u_hi = kept_t + pos_last / AM_KT - t_lo; // inclusive
     if (DECODE && ap.splits > 1) {
-        const int nt = t_hi - t_lo + 1, per = (nt + ap.splits - 1) / ap.splits;
-        t_lo += split * per;
-        if (t_lo + per - 1 < t_hi) t_hi = t_lo + per - 1;
+        const int per = (u_hi + ap.splits) / ap.splits;
+        u_lo = split * per;
+        if (u_lo + per - 1 < u_hi) u_hi = u_lo + per - 1;
     }
+    auto tile_of = [&](int u) { return u < kept_t ? u : u - kept_t + t_lo; };
     const size_t k_base = (size_t)kvh * pc.page_size * D.d, v_base = (size_t)D.G * pc.page_size * D.d + (size_t)kvh * pc.page_size * D.dv;
     const __nv_bfloat16* pool = (const __nv_bfloat16*)pc.pool + pc.layer_off;
     // a thread stages the same 16-byte column of every row it touches: 128 threads cover 128 / (row chunks) rows per pass
@@ -167,11 +172,11 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
     for (int j = 0; j < NVT; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
     const int kw0 = DECODE ? warp * 16 : 0;                // first key of the tile this warp consumes
 #pragma unroll
-    for (int i = 0; i < NSTAGE - 1; ++i) { if (t_lo + i <= t_hi) stage(t_lo + i, i); else am_commit(); }
-    for (int t = t_lo; t <= t_hi; ++t) {
-        const int buf = (t - t_lo) % NSTAGE;
+    for (int i = 0; i < NSTAGE - 1; ++i) { if (u_lo + i <= u_hi) stage(tile_of(u_lo + i), i); else am_commit(); }
+    for (int u = u_lo; u <= u_hi; ++u) {
+        const int buf = (u - u_lo) % NSTAGE;
         // the tile NSTAGE - 1 ahead goes into the buffer that the previous iteration finished reading (an empty group keeps the count uniform)
-        if (t + NSTAGE - 1 <= t_hi) stage(t + NSTAGE - 1, (t - t_lo + NSTAGE - 1) % NSTAGE); else am_commit();
+        if (u + NSTAGE - 1 <= u_hi) stage(tile_of(u + NSTAGE - 1), (u - u_lo + NSTAGE - 1) % NSTAGE); else am_commit();
         am_wait<NSTAGE - 1>();
         __syncthreads();
         // values that are the keys are read from the staged key tile itself (same row stride: DKP == DVP then)
@@ -196,13 +201,14 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
         // ---- distance penalty, mask, online softmax (rows g4 and g4 + 8 of the warp; a row's 4 lanes share it).  Scores are kept in
         // units of log 2 (scale and slope carry log2 e), so the exponentials are exp2.  The penalty of element (row, key) is
         // slope * (pos_row - key) = slope * (pos_row - jt0 - 2 t4) - slope * (column constant): one term per row and tile, one FMA per element.
-        const int jt0 = t * AM_KT + kw0;
+        const int jt0 = tile_of(u) * AM_KT + kw0;
         float nb[2];
 #pragma unroll
         for (int k = 0; k < 2; ++k) nb[k] = -r_slope2[k] * (float)(r_pos[k] - jt0 - 2 * t4);
         float mx[2] = {-INFINITY, -INFINITY};
-        // a tile every row of the warp sees whole needs no mask: its last key is not after the warp's first position, its first not before the window
-        const bool whole = jt0 + KW - 1 <= wpos_min && jt0 >= wlo_max;
+        // a tile every row of the warp sees whole needs no mask: its last key is not after the warp's first position, its first not before the
+        // window (or its last among the kept first ones)
+        const bool whole = jt0 + KW - 1 <= wpos_min && (jt0 >= wlo_max || jt0 + KW <= D.keep_first);
         if (EXT) {
 #pragma unroll
             for (int j = 0; j < NST; ++j)
@@ -210,7 +216,7 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
                 for (int e = 0; e < 4; ++e) {
                     const int k = e >> 1, key = jt0 + j * 8 + 2 * t4 + (e & 1);
                     const int dist = r_pos[k] - key;
-                    const bool vis = whole || (r_ok[k] && dist >= 0 && key >= r_lo[k]);
+                    const bool vis = whole || (r_ok[k] && dist >= 0 && (key >= r_lo[k] || key < D.keep_first));
                     float v = s[j][e] * D.scale;
                     // cap * tanh(v / cap) as cap * (1 - 2 / (exp(2 v / cap) + 1)): the hardware exponential and reciprocal keep the
                     // score to a few 1e-6 of the cap, well inside what the bf16 operands of the product leave
@@ -239,7 +245,7 @@ __global__ void __launch_bounds__(AM_THREADS, 3) gqa_attn_mma_kernel(Batch b, Gq
                 for (int e = 0; e < 4; ++e) {
                     const int k = e >> 1, key = jt0 + j * 8 + 2 * t4 + (e & 1);
                     const int dist = r_pos[k] - key;
-                    const bool vis = r_ok[k] && dist >= 0 && key >= r_lo[k];
+                    const bool vis = r_ok[k] && dist >= 0 && (key >= r_lo[k] || key < D.keep_first);
                     const float v = vis ? fmaf(s[j][e], scale2, fmaf(r_slope2[k], (float)(j * 8 + (e & 1)), nb[k])) : -INFINITY;
                     s[j][e] = v;
                     mx[k] = fmaxf(mx[k], v);
@@ -423,7 +429,7 @@ bool gqa_attn_mma_usable(const GqaDims& D, const PagedCache& pc) {
            ((long long)pc.page_size * D.d) % 8 == 0 && D.G <= 65535;
 }
 
-bool gqa_attn_mma_takes(const GqaDims& D) { return D.chunk >= 0 && D.softcap >= 0.f && !D.talk; }
+bool gqa_attn_mma_takes(const GqaDims& D) { return D.chunk >= 0 && D.softcap >= 0.f && !D.talk && !(D.keep_first > 0 && D.chunk > 0); }
 
 size_t gqa_attn_mma_workspace(int rows, int splits, int dv) { return (size_t)rows * splits * (dv + 2) * sizeof(float); }
 

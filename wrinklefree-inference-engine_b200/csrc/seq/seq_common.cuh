@@ -52,6 +52,11 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     __syncthreads();
     return scratch[32];
 }
+__device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
+__device__ __forceinline__ float epilogue_f(int ep, float v) {        // GemmArgs::ep
+    if (ep == 1) { v = fmaxf(v, 0.f); return v * v; }
+    return ep == 2 ? gelu_erf_f(v) : v;
+}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }

@@ -76,6 +76,8 @@ struct LayerState {
     // gated linear attention: decay bias
     void *r1_raw = nullptr, *r2_raw = nullptr, *talk_raw = nullptr, *a2_bias = nullptr;
     float *r1_f = nullptr, *r2_f = nullptr, *talk_f = nullptr;
+    // element-wise norms: before and behind the mixer, before and behind the feed-forward
+    DynNorm dn1, dn1b, dn2, dn2b;
     // state slot offsets (floats)
     size_t st_canon1 = 0, st_canon2 = 0, st_conv = 0, st_S = 0;
 };
@@ -91,6 +93,8 @@ struct wf_seq_engine {
     std::vector<TensorSlot> tensors;
     std::map<std::string, int> tensor_index;
     void *embed = nullptr, *final_norm = nullptr, *head = nullptr, *pos_table = nullptr, *final_norm_b = nullptr;
+    DynNorm final_dyn;
+    std::vector<char> again;          // per layer run: the embedding is added to the stream right before it (a repeated pass of the loop starts here)
     bool finalized = false;
     // cache + state
     PageTable pt;
@@ -174,7 +178,16 @@ void* at(const wf_seq_engine* e, void* base, size_t elems) { return (char*)base 
 
 int validate(const wf_seq_config& c, const wf_seq_layer* L) {
     if (c.dtype != WF_SEQ_F32 && c.dtype != WF_SEQ_BF16) { set_error("wf_seq_create: dtype %d", c.dtype); return WF_ERR_INVALID; }
-    if (c.vocab <= 0 || c.width <= 0 || c.n_layers <= 0 || c.norm_groups <= 0 || c.width % c.norm_groups || c.canon_taps < 1) {
+    const bool dyn = c.norm_kind == WF_SEQ_NORM_DYN_TANH;
+    if (c.norm_kind != WF_SEQ_NORM_RMS && !dyn) { set_error("wf_seq_create: norm kind %d", c.norm_kind); return WF_ERR_INVALID; }
+    if (dyn && (c.block_form != WF_SEQ_BLOCK_SANDWICH || c.canon_taps != 0 || c.pos_embed != 0 || c.norm_offset != 0.f)) {
+        set_error("wf_seq_create: element-wise norms belong to the sandwich form without input convolution, position embedding and weight offset"); return WF_ERR_UNSUPPORTED;
+    }
+    if (c.loop_times < 0 || (c.loop_times > 1 && (c.loop_start < 0 || c.loop_stop <= c.loop_start || c.loop_stop > c.n_layers))) {
+        set_error("wf_seq_create: layers %d .. %d of %d, %d times", c.loop_start, c.loop_stop, c.n_layers, c.loop_times); return WF_ERR_INVALID;
+    }
+    if (c.loop_times > 1 && !dyn) { set_error("wf_seq_create: repeated layers belong to the form with element-wise norms"); return WF_ERR_UNSUPPORTED; }
+    if (c.vocab <= 0 || c.width <= 0 || c.n_layers <= 0 || c.norm_groups <= 0 || c.width % c.norm_groups || (c.canon_taps < 1 && !dyn)) {
         set_error("wf_seq_create: vocab %d width %d layers %d norm groups %d taps %d", c.vocab, c.width, c.n_layers, c.norm_groups, c.canon_taps);
         return WF_ERR_INVALID;
     }
@@ -204,10 +217,13 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
                 set_error("layer %d: its second mixer differs in shape from that of layer %d", i, l.tied_to); return WF_ERR_INVALID;
             }
         }
+        if ((l.type == WF_SEQ_LATENT_ATTENTION || l.type == WF_SEQ_GQA_ATTENTION) &&
+            (l.rope_factor < 0.f || (l.rope_factor > 0.f && !(l.rope_orig > 0.f && l.rope_fast > 0.f && l.rope_slow > 0.f && l.rope_base > 1.f)))) {
+            set_error("layer %d: frequency interpolation constants", i); return WF_ERR_INVALID;
+        }
         if (l.type == WF_SEQ_LATENT_ATTENTION) {
             if (l.kv_rank <= 0 || l.rot_dim < 0 || l.window < 1 || l.rope_dims < 0 || l.rope_dims > l.rot_dim || (l.rope_dims & 1) || l.q_rank < 0) { set_error("layer %d: latent attention sizes", i); return WF_ERR_INVALID; }
             if (l.sink != 0 && l.sink != 2) { set_error("layer %d: latent attention takes no sink or a learned one per head", i); return WF_ERR_INVALID; }
-            if (l.rope_factor < 0.f || (l.rope_factor > 0.f && !(l.rope_orig > 0.f && l.rope_fast > 0.f && l.rope_slow > 0.f && l.rope_base > 1.f))) { set_error("layer %d: frequency interpolation constants", i); return WF_ERR_INVALID; }
         } else if (l.type == WF_SEQ_MINGRU) {
             if (l.heads != 1 || l.dim != 1) { set_error("layer %d: the element-wise recurrence has heads = dim = 1 and vdim channels", i); return WF_ERR_INVALID; }
         } else if (l.type == WF_SEQ_MLSTM) {
@@ -220,6 +236,8 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
             if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.conv < 1 || l.out_norm_groups < 1 || (l.heads * l.vdim) % l.out_norm_groups) { set_error("layer %d: state-space sizes", i); return WF_ERR_INVALID; }
         } else if (l.type == WF_SEQ_GQA_ATTENTION) {
             if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.window < 1) { set_error("layer %d: attention sizes", i); return WF_ERR_INVALID; }
+            if (l.v_is_k < 0 || l.v_is_k > 2 || l.keep_first < 0) { set_error("layer %d: value kind %d, %d kept first positions", i, l.v_is_k, l.keep_first); return WF_ERR_INVALID; }
+            if (l.keep_first > 0 && (l.chunk > 0 || l.talk)) { set_error("layer %d: kept first positions do not go with chunks or mixed heads", i); return WF_ERR_UNSUPPORTED; }
             if (l.v_is_k && (l.vdim != l.dim || l.v_norm || l.kv_from >= 0)) { set_error("layer %d: values that are the keys have the keys' size, no norm of their own and a cache of their own", i); return WF_ERR_INVALID; }
             if (l.sink < 0 || l.sink > 2) { set_error("layer %d: sink kind %d", i, l.sink); return WF_ERR_INVALID; }
             if (l.qk_norm < 0 || l.qk_norm > 3 || l.rope_dims < 0 || (l.rope_dims & 1) || l.rope_dims > l.dim || l.chunk < 0 || l.rel_rows < 0 || l.softcap < 0.f ||
@@ -238,9 +256,8 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
         if (l.pair_norm && !l.pair) { set_error("layer %d: output norms of a pair without a second mixer", i); return WF_ERR_INVALID; }
         if (l.has_ff != WF_SEQ_FF_NONE && l.has_ff != WF_SEQ_FF_ROUTED && l.has_ff != WF_SEQ_FF_DENSE) { set_error("layer %d: feed-forward kind %d", i, l.has_ff); return WF_ERR_INVALID; }
         if (l.has_ff == WF_SEQ_FF_DENSE && l.ff <= 0) { set_error("layer %d: dense feed-forward size", i); return WF_ERR_INVALID; }
-        if (l.ff_act == WF_SEQ_ACT_RELU2 && l.has_ff != WF_SEQ_FF_DENSE && l.has_ff != WF_SEQ_FF_NONE) { set_error("layer %d: the ungated activation belongs to a dense feed-forward", i); return WF_ERR_INVALID; }
         if (c.block_form == WF_SEQ_BLOCK_PARALLEL && l.has_ff == WF_SEQ_FF_ROUTED) { set_error("layer %d: the parallel block form takes a dense feed-forward or none", i); return WF_ERR_UNSUPPORTED; }
-        if (l.has_ff && (l.ff_act < 0 || l.ff_act > 3 || l.shared_ff < 0)) { set_error("layer %d: feed-forward activation / shared size", i); return WF_ERR_INVALID; }
+        if (l.has_ff && (l.ff_act < 0 || l.ff_act > WF_SEQ_ACT_GELU_ERF || l.shared_ff < 0)) { set_error("layer %d: feed-forward activation / shared size", i); return WF_ERR_INVALID; }
         if (l.has_ff == WF_SEQ_FF_ROUTED) {
             const int N = l.experts + l.identity;
             if (l.experts < 0 || l.identity < 0 || N <= 0 || l.top < 1 || l.top > N || l.groups < 1 || N % l.groups || l.keep < 1 || l.keep > l.groups || (l.experts > 0 && l.ff <= 0)) {
@@ -249,6 +266,48 @@ int validate(const wf_seq_config& c, const wf_seq_layer* L) {
         }
     }
     return WF_OK;
+}
+
+// A configuration with a loop, written out: one layer entry per run, later passes tied to the first one's weights.  ckpt: the layer whose
+// tensors a run uses; again: the run opens a repeated pass.
+struct Unrolled {
+    wf_seq_config cfg;
+    std::vector<wf_seq_layer> layers;
+    std::vector<int> ckpt;
+    std::vector<char> again;
+};
+Unrolled unroll(const wf_seq_config& c, const wf_seq_layer* L) {
+    Unrolled u;
+    u.cfg = c;
+    const int n = c.n_layers, a = c.loop_start, b = c.loop_stop, times = c.loop_times > 1 ? c.loop_times : 1, span = times > 1 ? b - a : 0, more = (times - 1) * span;
+    std::vector<int> pass;                                 // of every run
+    for (int i = 0; i < n; ++i) {
+        u.ckpt.push_back(i); pass.push_back(0);
+        if (span && i == b - 1)
+            for (int t = 1; t < times; ++t)
+                for (int j = a; j < b; ++j) { u.ckpt.push_back(j); pass.push_back(t); }
+    }
+    u.cfg.n_layers = n + more;
+    u.cfg.loop_times = 0;
+    auto first_run = [&](int layer) { return span && layer >= b ? layer + more : layer; };
+    std::vector<wf_seq_layer> extra(L + n, L + n + c.n_extra);
+    for (auto& m : extra) if (m.kv_from >= 0) m.kv_from = first_run(m.kv_from);
+    for (int r = 0; r < u.cfg.n_layers; ++r) {
+        const int i = u.ckpt[r];
+        wf_seq_layer l = L[i];
+        if (l.tied) l.tied_to = first_run(l.tied_to);
+        if (l.kv_from >= 0) l.kv_from = span && l.kv_from >= a && l.kv_from < b ? l.kv_from + (i >= b ? times - 1 : pass[r]) * span : first_run(l.kv_from);   // the same pass's rows; behind the loop, the last pass's
+        if (pass[r] > 0 && !l.tied) { l.tied = 1; l.tied_to = i; }
+        if (l.pair) {
+            if (pass[r] > 0) { extra.push_back(L[l.pair]); l.pair = u.cfg.n_layers + (int)extra.size() - 1; }
+            else l.pair += more;
+        }
+        u.layers.push_back(l);
+        u.again.push_back(pass[r] > 0 && i == a);
+    }
+    u.cfg.n_extra = (int)extra.size();
+    u.layers.insert(u.layers.end(), extra.begin(), extra.end());
+    return u;
 }
 
 void mark(wf_seq_engine* e, const char* label) {
@@ -474,7 +533,13 @@ int run_ssd(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     return rc;
 }
 
-// h_t -> y float [n, W].  In the post form the output projection's bias is NOT added here: the norm kernel that follows takes it
+// the output projection's bias is left to the norm kernel behind the mixer: the single-gain norm of the post form and the element-wise norms
+// take it, except for paired mixers (their outputs are combined first)
+bool norm_takes_bias(const wf_seq_engine* e, const LayerState& L) {
+    return !L.c.pair && (e->cfg.norm_kind == WF_SEQ_NORM_DYN_TANH || (e->cfg.block_form == WF_SEQ_BLOCK_POST && !e->cfg.norm_weights));
+}
+
+// h_t -> y float [n, W]; the output projection's bias only where the norm behind does not take it
 int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     const wf_seq_layer& c = L.c;
     const int W = e->cfg.width, n = b.n, nv = c.heads * c.vdim;
@@ -484,7 +549,8 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     D.rope_dims = c.rope_dims; D.rope_interleaved = c.rope_interleaved; D.rope_base = c.rope_base;
     D.q_norm_w = L.q_norm_w; D.k_norm_w = L.k_norm_w;
     D.chunk = c.chunk; D.sink = c.sink; D.gate_elem = c.head_gate == 2; D.softcap = c.softcap;
-    D.rel = L.rel_dist; D.rel_n = L.rel_n; D.v_is_k = c.v_is_k;
+    D.rel = L.rel_dist; D.rel_n = L.rel_n; D.v_is_k = c.v_is_k == 1;
+    D.keep_first = c.keep_first; D.freq = L.freq; D.mscale = L.rope_mscale;
     D.dist_r1 = L.r1_f; D.dist_r2 = L.r2_f; D.sink_h = L.sink_f; D.talk = L.talk_f;
     const LayerState& src = c.kv_from >= 0 ? e->layers[c.kv_from] : L;        // whose cache rows this layer reads
     PagedCache pc{e->pool, e->page_stride, src.cache_off, e->cfg.page_size, e->d_block_table, e->pt.max_blocks};
@@ -492,12 +558,12 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     int ld;
     if ((rc = in_proj(e, L, b, &pj, &ld))) return rc;     // [q | k | v | g]
     mark(e, "attn.proj_gemm");
-    if ((rc = launch_gqa_prep(e->dt, b, D, pj, ld, L.k_off, L.v_off, L.g_off, L.qb, L.kb, L.vb, e->cfg.eps, pc, e->qn, c.head_gate ? e->gate : nullptr, s))) return rc;
+    if ((rc = launch_gqa_prep(e->dt, b, D, pj, ld, L.k_off, c.v_is_k == 2 ? L.k_off : L.v_off, L.g_off, L.qb, L.kb, c.v_is_k == 2 ? L.kb : L.vb, e->cfg.eps, pc, e->qn, c.head_gate ? e->gate : nullptr, s))) return rc;
     mark(e, "attn.prep+kv_write");
     const float* gate = c.head_gate ? e->gate : nullptr;
     // decoding (one token per sequence) cuts the key range over blocks; the cut depends on the batch size and the pool only, never on the
     // lengths: a captured step stays valid
-    long long span = std::min<long long>(c.window, (long long)e->cfg.max_pages * e->cfg.page_size);
+    long long span = std::min<long long>((long long)c.window + c.keep_first, (long long)e->cfg.max_pages * e->cfg.page_size);
     if (c.chunk > 0 && c.chunk < span) span = c.chunk;
     if (e->dt == WF_BF16 && e->attn_mma >= 1 && D.talk && !gate && talk_attn_mma_usable(D, pc)) {
         int splits = 1;
@@ -525,8 +591,7 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
     } else if ((rc = launch_gqa_attn(e->dt, b, D, e->qn, gate, pc, e->og, s))) return rc;
     mark(e, D.talk ? "attn.attention(mixed heads)" : D.softcap > 0.f || D.rel ? "attn.attention(cap+bias)" : "attn.attention");
     rc = launch_gemm(e->dt, lin(e->og, 0, nv, L.wo, nv, out, 1, W, n, W, nv), s);
-    // the single-gain norm of the post form takes the bias itself, except for paired mixers (their outputs are combined first)
-    if (!rc && L.ob && !(e->cfg.block_form == WF_SEQ_BLOCK_POST && !e->cfg.norm_weights && !L.c.pair && out == e->y)) rc = launch_add_bias(e->dt, out, W, L.ob, n, W, s);
+    if (!rc && L.ob && !(norm_takes_bias(e, L) && out == e->y)) rc = launch_add_bias(e->dt, out, W, L.ob, n, W, s);
     mark(e, "attn.out_gemm");
     return rc;
 }
@@ -627,37 +692,52 @@ int run_mixer(wf_seq_engine* e, LayerState& L, const Batch& b, bool combine = tr
     return rc;
 }
 
-// the gated unit every token runs (dense feed-forward / shared expert): h_t -> out float [n, W]
+// activations without a gate half are formed where the product stores its results
+int ungated_ep(int act) { return act == WF_SEQ_ACT_RELU2 ? EP_RELU2 : act == WF_SEQ_ACT_GELU_ERF ? EP_GELU_ERF : EP_NONE; }
+
+// the unit every token runs (dense feed-forward / shared expert): h_t -> out float [n, W]
 int run_unit(wf_seq_engine* e, LayerState& L, const Batch& b, float* out, const void* in = nullptr) {
     const int W = e->cfg.width, n = b.n, ff = L.uff;
     cudaStream_t s = e->stream;
     int rc;
     if (!in) in = e->h_t;
-    const int nu = L.c.ff_act == WF_SEQ_ACT_RELU2 ? ff : 2 * ff;       // the ungated activation has no gate half
-    if ((rc = launch_gemm(e->dt, lin(in, 0, W, L.ugu, W, e->ugu, 1, nu, n, nu, W), s))) return rc;
-    mark(e, "unit.gate_up");
-    if ((rc = launch_silu_mul(e->dt, e->ugu, n, ff, nullptr, e->uhmid, s, L.c.ff_act, L.ulimit))) return rc;
-    mark(e, "unit.act");
+    if (const int ep = ungated_ep(L.c.ff_act)) {
+        GemmArgs g = lin(in, 0, W, L.ugu, W, e->uhmid, 0, ff, n, ff, W);
+        g.ep = ep;
+        if ((rc = launch_gemm(e->dt, g, s))) return rc;
+        mark(e, "unit.up");
+    } else {
+        if ((rc = launch_gemm(e->dt, lin(in, 0, W, L.ugu, W, e->ugu, 1, 2 * ff, n, 2 * ff, W), s))) return rc;
+        mark(e, "unit.gate_up");
+        if ((rc = launch_silu_mul(e->dt, e->ugu, n, ff, nullptr, e->uhmid, s, L.c.ff_act, L.ulimit))) return rc;
+        mark(e, "unit.act");
+    }
     rc = launch_gemm(e->dt, lin(e->uhmid, 0, ff, L.ud, ff, out, 1, W, n, W, ff), s);
     mark(e, "unit.down");
     return rc;
 }
 
-int run_ff(wf_seq_engine* e, LayerState& L, const Batch& b) {
+// st (optional): the stream update that follows takes the feed-forward's output, or the routed experts' outputs and weights, from there
+int run_ff(wf_seq_engine* e, LayerState& L, const Batch& b, StreamStep* st = nullptr) {
     const wf_seq_layer& c = L.c;
     const int W = e->cfg.width, n = b.n, N = L.nz;
     cudaStream_t s = e->stream;
     int rc;
-    if (c.has_ff == WF_SEQ_FF_DENSE) return run_unit(e, L, b, e->y);
+    if (c.has_ff == WF_SEQ_FF_DENSE) {
+        if (st) st->y = e->y;
+        return run_unit(e, L, b, e->y);
+    }
     RouterDims R{c.experts, c.identity, c.top, c.groups, c.keep};
     R.act = c.router_act; R.group_top = c.group_top; R.norm = c.router_norm; R.scale = c.router_scale != 0.f ? c.router_scale : 1.f;   // a zeroed struct means unscaled
-    // In the post form the sublayer's input IS the float stream, so the router reads it unrounded and multiplies in float — a router is
-    // a 32-bit quantity, and a score that the rounding of its input moved across a neighbour's would change the chosen experts — and the
-    // product and the choice are one kernel.  The sandwich form's input exists only in the storage type: product, then choice.
-    const bool fused_router = e->cfg.block_form == WF_SEQ_BLOCK_POST && router_fused_usable(R, N, W);
+    // In the post form the sublayer's input IS the float stream, and element-wise norms leave a float copy of it (hn), so the router reads
+    // it unrounded and multiplies in float — a router is a 32-bit quantity, and a score that the rounding of its input moved across a
+    // neighbour's would change the chosen experts — and the product and the choice are one kernel.  Behind an input convolution the input
+    // exists only in the storage type: product, then choice.
+    const float* rx = e->cfg.norm_kind == WF_SEQ_NORM_DYN_TANH ? e->hn : e->cfg.block_form == WF_SEQ_BLOCK_POST ? e->x : nullptr;
+    const bool fused_router = rx && router_fused_usable(R, N, W);
     if (!fused_router) {
-        GemmArgs g = e->cfg.block_form == WF_SEQ_BLOCK_POST ? lin(e->x, 1, W, L.router, W, e->z, 1, N, n, N, W) : lin(e->h_t, 0, W, L.router, W, e->z, 1, N, n, N, W);
-        if (e->cfg.block_form == WF_SEQ_BLOCK_POST && (n > 8 || W % 8)) g.algo = 1;      // up to 8 aligned rows take the few-row stream, which multiplies in float too
+        GemmArgs g = rx ? lin(rx, 1, W, L.router, W, e->z, 1, N, n, N, W) : lin(e->h_t, 0, W, L.router, W, e->z, 1, N, n, N, W);
+        if (rx && (n > 8 || W % 8)) g.algo = 1;      // up to 8 aligned rows take the few-row stream, which multiplies in float too
         if ((rc = launch_gemm(e->dt, g, s))) return rc;     // expert logits [| shared gate logit]
         mark(e, "moe.router");
     }
@@ -665,28 +745,34 @@ int run_ff(wf_seq_engine* e, LayerState& L, const Batch& b) {
     const float* sh_gate = nullptr;
     if (c.shared_ff > 0) {
         if ((rc = run_unit(e, L, b, e->uy))) return rc;
-        sh_y = e->uy; sh_gate = e->z + c.experts + c.identity;
+        sh_y = e->uy;
+        if (!c.shared_plain) sh_gate = e->z + c.experts + c.identity;
     }
     const int pairs = n * c.top;
-    GemmArgs gp = lin(e->h_t, 0, W, L.wgu, W, e->gu, 1, 2 * c.ff, pairs, 2 * c.ff, W);
-    gp.group_stride = (long long)2 * c.ff * W;
+    const int ep = ungated_ep(c.ff_act), nu = ep ? c.ff : 2 * c.ff;          // rows of an expert's input matrix
+    GemmArgs gp = ep ? lin(e->h_t, 0, W, L.wgu, W, e->hmid, 0, nu, pairs, nu, W) : lin(e->h_t, 0, W, L.wgu, W, e->gu, 1, nu, pairs, nu, W);
+    gp.group_stride = (long long)nu * W; gp.ep = ep;
     GemmArgs gd = lin(e->hmid, 0, c.ff, L.wd, c.ff, e->yexp, 1, W, pairs, W, c.ff);
     gd.group_stride = (long long)W * c.ff;
+    const bool combine_later = st && c.identity == 0 && !sh_gate;
     const bool pair_path = c.experts > 0 && pairs <= e->pair_path_max && gemv_pairs_usable(e->dt, gp) && gemv_pairs_usable(e->dt, gd);
     // per-expert token counts are only needed to sort the pairs (the per-pair path sorts nothing)
     if (c.experts > 0 && !pair_path && cuda_check(cudaMemsetAsync(e->counts, 0, (size_t)c.experts * 4, s), "counts")) return WF_ERR_CUDA;
-    if (fused_router) rc = launch_router_fused(e->dt, R, n, e->x, W, L.router, N, W, e->z, N, L.correction, e->ids, e->wts, pair_path ? nullptr : e->counts, s);
+    if (fused_router) rc = launch_router_fused(e->dt, R, n, rx, W, L.router, N, W, e->z, N, L.correction, e->ids, e->wts, pair_path ? nullptr : e->counts, s);
     else rc = launch_moe_route(e->dt, R, n, e->z, N, L.correction, e->ids, e->wts, pair_path ? nullptr : e->counts, s);
     if (rc) return rc;
     mark(e, "moe.router");
     if (pair_path) {
         // few tokens (decoding): one weight-streaming product per (token, expert) pair, no sorting
         if ((rc = launch_gemv_pairs(e->dt, gp, e->ids, c.experts, pairs, c.top, s))) return rc;
-        mark(e, "moe.gate_up");
-        if ((rc = launch_silu_mul(e->dt, e->gu, pairs, c.ff, nullptr, e->hmid, s, c.ff_act, c.ff_limit))) return rc;
-        mark(e, "moe.silu_mul");
+        mark(e, ep ? "moe.up" : "moe.gate_up");
+        if (!ep) {
+            if ((rc = launch_silu_mul(e->dt, e->gu, pairs, c.ff, nullptr, e->hmid, s, c.ff_act, c.ff_limit))) return rc;
+            mark(e, "moe.silu_mul");
+        }
         if ((rc = launch_gemv_pairs(e->dt, gd, e->ids, c.experts, pairs, 1, s))) return rc;
         mark(e, "moe.down");
+        if (combine_later) { st->yexp = e->yexp; st->wts = e->wts; st->top = c.top; st->shared_y = sh_y; return WF_OK; }
         rc = launch_moe_combine(e->dt, R, n, W, e->ids, e->wts, nullptr, e->yexp, e->h_t, e->y, s, sh_y, sh_gate, N);
         mark(e, "moe.combine");
         return rc;
@@ -697,17 +783,21 @@ int run_ff(wf_seq_engine* e, LayerState& L, const Batch& b) {
         mark(e, "moe.plan");
         // the experts' input rows, expert after expert (a dense operand for the tensor-core product)
         if ((rc = launch_gather_rows(e->dt, e->h_t, W, e->sorted_rows, P, W, e->hperm, s))) return rc;
-        GemmArgs g = lin(e->hperm, 0, W, L.wgu, W, e->gu, 1, 2 * c.ff, P, 2 * c.ff, W);
-        g.tile_group = e->tile_group; g.group_stride = (long long)2 * c.ff * W; g.n_groups = c.experts;
+        GemmArgs g = ep ? lin(e->hperm, 0, W, L.wgu, W, e->hmid, 0, nu, P, nu, W) : lin(e->hperm, 0, W, L.wgu, W, e->gu, 1, nu, P, nu, W);
+        g.tile_group = e->tile_group; g.group_stride = (long long)nu * W; g.n_groups = c.experts; g.ep = ep;
         if ((rc = launch_gemm(e->dt, g, s))) return rc;
-        mark(e, "moe.gate_up");
-        if ((rc = launch_silu_mul(e->dt, e->gu, P, c.ff, e->tile_group, e->hmid, s, c.ff_act, c.ff_limit))) return rc;
-        mark(e, "moe.silu_mul");
+        mark(e, ep ? "moe.up" : "moe.gate_up");
+        if (!ep) {
+            if ((rc = launch_silu_mul(e->dt, e->gu, P, c.ff, e->tile_group, e->hmid, s, c.ff_act, c.ff_limit))) return rc;
+            mark(e, "moe.silu_mul");
+        }
         GemmArgs g2 = lin(e->hmid, 0, c.ff, L.wd, c.ff, e->yexp, 1, W, P, W, c.ff);
         g2.tile_group = e->tile_group; g2.group_stride = (long long)W * c.ff; g2.n_groups = c.experts;
         if ((rc = launch_gemm(e->dt, g2, s))) return rc;
         mark(e, "moe.down");
     }
+    if (combine_later) { st->yexp = e->yexp; st->wts = e->wts; st->pair_row = e->pair_row; st->top = c.top; st->shared_y = sh_y; return WF_OK; }
+    if (st) st->y = e->y;
     rc = launch_moe_combine(e->dt, R, n, W, e->ids, e->wts, e->pair_row, e->yexp, e->h_t, e->y, s, sh_y, sh_gate, N);
     mark(e, "moe.combine");
     return rc;
@@ -834,7 +924,48 @@ int run_layers_one_norm(wf_seq_engine* e, const StepView& v) {
     return WF_OK;
 }
 
+// The sandwich form with element-wise norms and no input convolution: one kernel between two sublayers forms a sublayer's output norm (of
+// routed experts: their weighted sum first), adds it to the stream, adds the embedding where a repeated pass begins, and leaves the next
+// sublayer's normed input.
+int run_layers_dyn(wf_seq_engine* e, const StepView& v) {
+    const int W = e->cfg.width, n = v.b.n, NL = e->cfg.n_layers;
+    cudaStream_t s = e->stream;
+    int rc;
+    const float escale = e->cfg.embed_scale != 0.f ? e->cfg.embed_scale : 1.f;
+    StreamStep first;
+    first.init = 1; first.embed = e->embed; first.tokens = v.tokens; first.embed_scale = escale; first.pre = e->layers[0].dn1; first.h = e->h_t;
+    if ((rc = launch_stream_step(e->dt, e->x, first, n, W, s))) return rc;
+    mark(e, "embed+norm");
+    for (int li = 0; li < NL; ++li) {
+        LayerState& L = e->layers[li];
+        if ((rc = run_mixer(e, L, v.b))) return rc;
+        StreamStep st;
+        st.y = e->y; st.bias = norm_takes_bias(e, L) ? L.ob : nullptr; st.post = L.dn1b;
+        if (L.c.has_ff) {
+            st.pre = L.dn2; st.h = e->h_t; st.hf = L.c.has_ff == WF_SEQ_FF_ROUTED ? e->hn : nullptr;
+            if ((rc = launch_stream_step(e->dt, e->x, st, n, W, s))) return rc;
+            mark(e, "norms+residual");
+            st = StreamStep();
+            if ((rc = run_ff(e, L, v.b, &st))) return rc;
+            st.post = L.dn2b;
+        }
+        if (e->layer_tap) {                  // the stream as this layer leaves it, before what belongs to the next one
+            if ((rc = launch_stream_step(e->dt, e->x, st, n, W, s))) return rc;
+            if (cuda_check(cudaMemcpyAsync(e->layer_tap + (size_t)li * n * W, e->x, (size_t)n * W * 4, cudaMemcpyDeviceToHost, s), "layer tap")) return WF_ERR_CUDA;
+            st = StreamStep();
+        }
+        if (li + 1 < NL) {
+            st.pre = e->layers[li + 1].dn1; st.h = e->h_t;
+            if (e->again[li + 1]) { st.embed = e->embed; st.tokens = v.tokens; st.embed_scale = escale; }
+        } else if (e->layer_tap) break;
+        if ((rc = launch_stream_step(e->dt, e->x, st, n, W, s))) return rc;
+        mark(e, "norms+residual");
+    }
+    return WF_OK;
+}
+
 int run_layers(wf_seq_engine* e, const StepView& v) {
+    if (e->cfg.norm_kind == WF_SEQ_NORM_DYN_TANH) return run_layers_dyn(e, v);
     if (e->cfg.one_norm) return run_layers_one_norm(e, v);
     if (e->cfg.block_form == WF_SEQ_BLOCK_POST) return run_layers_post(e, v);
     if (e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL) return run_layers_parallel(e, v);
@@ -878,7 +1009,8 @@ int run_head(wf_seq_engine* e, const StepView& v, int nwant) {
     const int W = e->cfg.width;
     int rc;
     if ((rc = ensure_logits(e, nwant))) return rc;
-    if (e->cfg.layer_norm) rc = launch_layer_norm(e->dt, e->x, W, e->final_norm, e->final_norm_b, e->cfg.eps, nwant, W, nullptr, W, e->xn, W, v.want, e->stream);
+    if (e->cfg.norm_kind == WF_SEQ_NORM_DYN_TANH) rc = launch_dyn_tanh(e->dt, e->x, W, e->final_dyn, nwant, W, nullptr, e->xn, v.want, e->stream);
+    else if (e->cfg.layer_norm) rc = launch_layer_norm(e->dt, e->x, W, e->final_norm, e->final_norm_b, e->cfg.eps, nwant, W, nullptr, W, e->xn, W, v.want, e->stream);
     else if (e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL) rc = launch_group_rmsnorm(e->dt, e->x, W, e->final_norm, 1, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream, nullptr, 1.f, 0.f, e->cfg.norm_offset);
     else if (e->cfg.block_form == WF_SEQ_BLOCK_POST && e->cfg.norm_weights) rc = launch_group_rmsnorm(e->dt, e->x, W, e->final_norm, 1, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream);
     else if (e->cfg.block_form == WF_SEQ_BLOCK_POST) rc = launch_scalar_rmsnorm(e->dt, e->x, W, nullptr, e->final_norm, 1.f, e->cfg.eps, nwant, W, nullptr, nullptr, W, e->xn, W, v.want, e->stream);
@@ -936,9 +1068,13 @@ extern "C" int wf_seq_available(void) {
 extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layers, wf_seq_engine** out) {
     if (!cfg || !layers || !out) { set_error("wf_seq_create: null argument"); return WF_ERR_INVALID; }
     if (int rc = validate(*cfg, layers)) return rc;
+    const Unrolled un = unroll(*cfg, layers);          // from here on a layer is a layer run
+    layers = un.layers.data();
+    if (int rc = validate(un.cfg, layers)) return rc;
     if (!wf_seq_available()) { set_error("wf_seq_create: no compute-capability-10.x device"); return WF_ERR_UNSUPPORTED; }
     wf_seq_engine* e = new wf_seq_engine();
-    e->cfg = *cfg;
+    e->cfg = un.cfg;
+    e->again = un.again;
     e->dt = cfg->dtype == WF_SEQ_F32 ? WF_F32 : WF_BF16;
     e->esz = e->dt == WF_F32 ? 4 : 2;
     if (const char* pm = getenv("WF_SEQ_PAIR_MAX")) e->pair_path_max = atoi(pm);
@@ -958,7 +1094,13 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
     TRY(dalloc_t(e, &e->final_norm, norm_elems));
     add_tensor(e, "embed", e->embed, (size_t)c.vocab * W);
     add_tensor(e, "final.norm", e->final_norm, norm_elems);
-    if (c.layer_norm) { TRY(dalloc_t(e, &e->final_norm_b, W)); add_tensor(e, "final.norm.b", e->final_norm_b, W); }
+    const bool dyn = c.norm_kind == WF_SEQ_NORM_DYN_TANH;
+    if (c.layer_norm || dyn) { TRY(dalloc_t(e, &e->final_norm_b, W)); add_tensor(e, "final.norm.b", e->final_norm_b, W); }
+    if (dyn) {
+        void* al = nullptr;
+        TRY(dalloc_t(e, &al, 1)); add_tensor(e, "final.norm.alpha", al, 1);
+        e->final_dyn.w = e->final_norm; e->final_dyn.b = e->final_norm_b; e->final_dyn.alpha = al;
+    }
     if (c.pos_embed == 2) { TRY(dalloc_t(e, &e->pos_table, (size_t)c.max_positions * W)); add_tensor(e, "pos", e->pos_table, (size_t)c.max_positions * W); }
     if (c.tied_head) e->head = e->embed;
     else { TRY(dalloc_t(e, &e->head, (size_t)c.vocab * W)); add_tensor(e, "head", e->head, (size_t)c.vocab * W); }
@@ -985,7 +1127,8 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
             const bool ownkv = l.kv_from < 0;
             const size_t ng = l.head_gate == 2 ? nv : (size_t)l.heads;
             size_t off = nq;
-            const bool ownv = ownkv && !l.v_is_k;       // values that are the keys are neither projected nor cached
+            const bool ownv = ownkv && !l.v_is_k;       // values that are the keys are not projected ...
+            const bool cachev = ownkv && l.v_is_k != 1; // ... nor, when they are the keys as cached, cached
             if (ownkv) { L.k_off = (int)off; off += nk; }
             if (ownv) { L.v_off = (int)off; off += nvk; }
             if (l.head_gate) { L.g_off = (int)off; off += ng; }
@@ -1010,6 +1153,7 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
                 TRYL(walloc(&L.q_norm_w, wq)); name(mp + "q.norm", L.q_norm_w, wq);
                 TRYL(walloc(&L.k_norm_w, wk)); name(mp + "k.norm", L.k_norm_w, wk);      // a layer that reads another's cache still names it: unused
             }
+            if (own && l.rope_dims > 0) TRYL(dalloc_n(e, &L.freq, l.rope_dims / 2));
             if (l.dist_log) {
                 TRYL(walloc(&L.r1_raw, l.heads)); name(mp + "r1", L.r1_raw, l.heads);
                 TRYL(walloc(&L.r2_raw, l.heads)); name(mp + "r2", L.r2_raw, l.heads);
@@ -1033,7 +1177,7 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
                 // every layer's part of a page starts 16-byte aligned
                 cache_elems = (cache_elems + 7) / 8 * 8;
                 L.cache_off = cache_elems;
-                cache_elems += (long long)c.page_size * (nk + (ownv ? nvk : 0));
+                cache_elems += (long long)c.page_size * (nk + (cachev ? nvk : 0));
             }
             if (l.talk) {
                 GqaDims T{l.heads, l.kv_heads, l.dim, l.vdim, 0.f, 0.f, 1, 0, 0};
@@ -1177,12 +1321,21 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
         if (!own) L = e->layers[layers[li].tied_to];      // the source's weight pointers; offsets of cache and state are assigned anew below
         L.c = layers[li];
         const wf_seq_layer& l = L.c;
-        const std::string p = "l" + std::to_string(li) + ".";
+        const std::string p = "l" + std::to_string(un.ckpt[li]) + ".";
         if (own) L.norm1 = L.norm2 = L.norm1b = L.norm2b = L.canon1 = L.canon2 = nullptr;
         if (post) {
             TRY(walloc(&L.norm1, lnorm)); name(p + "norm1", L.norm1, lnorm);
             if (c.layer_norm) { TRY(walloc(&L.norm1_bias, W)); name(p + "norm1.b", L.norm1_bias, W); }
             if (l.has_ff && !c.one_norm) { TRY(walloc(&L.norm2, lnorm)); name(p + "norm2", L.norm2, lnorm); }
+        } else if (dyn) {
+            DynNorm* norms[4] = {&L.dn1, &L.dn1b, &L.dn2, &L.dn2b};
+            const char* norm_names[4] = {"norm1", "norm1b", "norm2", "norm2b"};
+            for (int k = 0; k < (l.has_ff ? 4 : 2) && own; ++k) {
+                void *w = nullptr, *b = nullptr, *al = nullptr;
+                TRY(dalloc_t(e, &w, W)); TRY(dalloc_t(e, &b, W)); TRY(dalloc_t(e, &al, 1));
+                norms[k]->w = w; norms[k]->b = b; norms[k]->alpha = al;
+                name(p + norm_names[k], w, W); name(p + norm_names[k] + ".b", b, W); name(p + norm_names[k] + ".alpha", al, 1);
+            }
         } else {
             void** norms[4] = {&L.norm1, &L.norm1b, &L.norm2, &L.norm2b};
             const char* norm_names[4] = {"norm1", "norm1b", "norm2", "norm2b"};
@@ -1225,7 +1378,7 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
         max_np = std::max(max_np, (size_t)L.in_np);
         if (l.has_ff == WF_SEQ_FF_DENSE) {
             L.uff = l.ff; L.ulimit = l.ff_limit;
-            const bool gated = l.ff_act != WF_SEQ_ACT_RELU2;
+            const bool gated = !ungated_ep(l.ff_act);
             TRY(walloc(&L.ugu, (size_t)(gated ? 2 : 1) * l.ff * W)); TRY(walloc(&L.ud, (size_t)W * l.ff));
             if (gated) name(p + "mlp.gate", L.ugu, (size_t)l.ff * W);
             name(p + "mlp.up", at(e, L.ugu, gated ? (size_t)l.ff * W : 0), (size_t)l.ff * W);
@@ -1233,25 +1386,27 @@ extern "C" int wf_seq_create(const wf_seq_config* cfg, const wf_seq_layer* layer
             max_uff = std::max(max_uff, (size_t)l.ff);
         } else if (l.has_ff == WF_SEQ_FF_ROUTED) {
             const size_t N = l.experts + l.identity;
-            L.nz = (int)N + (l.shared_ff > 0 ? 1 : 0);
+            const bool gated = !ungated_ep(l.ff_act);
+            const size_t halves = gated ? 2 : 1;
+            L.nz = (int)N + (l.shared_ff > 0 && !l.shared_plain ? 1 : 0);
             TRY(walloc(&L.router, (size_t)L.nz * W)); name(p + "mlp.router", L.router, N * W);
             if (l.shared_ff > 0) {
                 L.uff = l.shared_ff; L.ulimit = l.shared_limit;
-                name(p + "mlp.shared.sg", at(e, L.router, N * W), W);
-                TRY(walloc(&L.ugu, (size_t)2 * l.shared_ff * W)); TRY(walloc(&L.ud, (size_t)W * l.shared_ff));
-                name(p + "mlp.shared.gate", L.ugu, (size_t)l.shared_ff * W);
-                name(p + "mlp.shared.up", at(e, L.ugu, (size_t)l.shared_ff * W), (size_t)l.shared_ff * W);
+                if (!l.shared_plain) name(p + "mlp.shared.sg", at(e, L.router, N * W), W);
+                TRY(walloc(&L.ugu, halves * l.shared_ff * W)); TRY(walloc(&L.ud, (size_t)W * l.shared_ff));
+                if (gated) name(p + "mlp.shared.gate", L.ugu, (size_t)l.shared_ff * W);
+                name(p + "mlp.shared.up", at(e, L.ugu, gated ? (size_t)l.shared_ff * W : 0), (size_t)l.shared_ff * W);
                 name(p + "mlp.shared.down", L.ud, (size_t)W * l.shared_ff);
                 max_uff = std::max(max_uff, (size_t)l.shared_ff);
             }
-            TRY(walloc(&L.correction, N)); name(p + "mlp.correction", L.correction, N);
+            if (!l.no_correction) { TRY(walloc(&L.correction, N)); name(p + "mlp.correction", L.correction, N); }
             if (l.experts > 0) {
-                TRY(walloc(&L.wgu, (size_t)l.experts * 2 * l.ff * W));
+                TRY(walloc(&L.wgu, (size_t)l.experts * halves * l.ff * W));
                 TRY(walloc(&L.wd, (size_t)l.experts * W * l.ff));
                 for (int x = 0; x < l.experts; ++x) {
                     const std::string ep = p + "mlp.e" + std::to_string(x) + ".";
-                    name(ep + "gate", at(e, L.wgu, (size_t)x * 2 * l.ff * W), (size_t)l.ff * W);
-                    name(ep + "up", at(e, L.wgu, ((size_t)x * 2 + 1) * l.ff * W), (size_t)l.ff * W);
+                    if (gated) name(ep + "gate", at(e, L.wgu, (size_t)x * 2 * l.ff * W), (size_t)l.ff * W);
+                    name(ep + "up", at(e, L.wgu, ((x + 1) * halves - 1) * l.ff * W), (size_t)l.ff * W);
                     name(ep + "down", at(e, L.wd, (size_t)x * W * l.ff), (size_t)W * l.ff);
                 }
             }
@@ -1331,6 +1486,7 @@ extern "C" void wf_seq_destroy(wf_seq_engine* e) {
 }
 
 extern "C" size_t wf_seq_device_bytes(const wf_seq_engine* e) { return e ? e->dev_bytes : 0; }
+extern "C" int wf_seq_layer_runs(const wf_seq_engine* e) { return e ? e->cfg.n_layers : 0; }
 extern "C" int wf_seq_tensor_count(const wf_seq_engine* e) { return e ? (int)e->tensors.size() : 0; }
 extern "C" const char* wf_seq_tensor_name(const wf_seq_engine* e, int i, size_t* count, int* loaded) {
     if (!e || i < 0 || i >= (int)e->tensors.size()) return nullptr;
@@ -1400,18 +1556,19 @@ extern "C" int wf_seq_finalize(wf_seq_engine* e) {
         if (cuda_check(cudaMemcpyAsync(L.rel_dist, tab.data(), tab.size() * 4, cudaMemcpyHostToDevice, e->stream), "bias table H2D")) return WF_ERR_CUDA;
         if (cuda_check(cudaStreamSynchronize(e->stream), "sync")) return WF_ERR_CUDA;
     }
-    // latent attention: the rotation's frequencies, tabulated in double (with frequency interpolation: pairs whose wavelength is long
+    // attention: the rotation's frequencies, tabulated in double (with frequency interpolation: pairs whose wavelength is long
     // against the original context turn `factor` times slower, short ones as they are, a linear ramp over the pair index between), and
     // the learned sinks as floats
     for (LayerState& L : e->layers) {
-        if (L.c.type != WF_SEQ_LATENT_ATTENTION || L.c.tied) continue;
+        if (L.c.type != WF_SEQ_LATENT_ATTENTION && L.c.type != WF_SEQ_GQA_ATTENTION) continue;
         const wf_seq_layer& l = L.c;
+        L.rope_mscale = l.rope_factor > 0.f ? (float)(0.1 * log((double)l.rope_factor) + 1.0) : 1.f;
+        if (l.tied) continue;                 // its source's table
         if (L.freq) {
             const int dims = l.rope_dims, half = dims / 2;
             const double base = l.rope_base, pi = 3.14159265358979323846;
             std::vector<double> f(half);
             for (int i = 0; i < half; ++i) f[i] = pow(base, -2.0 * i / dims);
-            L.rope_mscale = 1.f;
             if (l.rope_factor > 0.f) {
                 const double factor = l.rope_factor;
                 auto pair_of = [&](double turns) { return dims * log((double)l.rope_orig / (2.0 * pi * turns)) / (2.0 * log(base)); };
@@ -1420,25 +1577,23 @@ extern "C" int wf_seq_finalize(wf_seq_engine* e) {
                     const double ramp = std::min(std::max(((double)i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
                     f[i] = f[i] / factor * ramp + f[i] * (1.0 - ramp);
                 }
-                L.rope_mscale = (float)(0.1 * log(factor) + 1.0);
             }
             if (cuda_check(cudaMemcpyAsync(L.freq, f.data(), f.size() * sizeof(double), cudaMemcpyHostToDevice, e->stream), "rotation table H2D")) return WF_ERR_CUDA;
             if (cuda_check(cudaStreamSynchronize(e->stream), "sync")) return WF_ERR_CUDA;
         }
         if (int rc = to_floats(e, L.sink_raw, L.sink_f, l.heads)) return rc;
     }
-    // grouped-query attention: learned penalty numbers, sinks and head mixture as floats
+    // grouped-query attention: learned penalty numbers and head mixture as floats
     for (LayerState& L : e->layers) {
         if (L.c.type != WF_SEQ_GQA_ATTENTION || L.c.tied) continue;
         const size_t H = L.c.heads;
         if (int rc = to_floats(e, L.r1_raw, L.r1_f, H)) return rc;
         if (int rc = to_floats(e, L.r2_raw, L.r2_f, H)) return rc;
-        if (int rc = to_floats(e, L.sink_raw, L.sink_f, H)) return rc;
         if (int rc = to_floats(e, L.talk_raw, L.talk_f, H * H)) return rc;
     }
     // tied latent layers use their source's tables
     for (LayerState& L : e->layers)
-        if (L.c.type == WF_SEQ_LATENT_ATTENTION && L.c.tied) { const LayerState& S = e->layers[L.c.tied_to]; L.freq = S.freq; L.sink_f = S.sink_f; L.rope_mscale = S.rope_mscale; }
+        if (L.c.type == WF_SEQ_LATENT_ATTENTION && L.c.tied) { const LayerState& S = e->layers[L.c.tied_to]; L.freq = S.freq; L.sink_f = S.sink_f; }
     if (cuda_check(cudaStreamSynchronize(e->stream), "finalize")) return WF_ERR_CUDA;
     e->finalized = true;
     return WF_OK;
@@ -1518,9 +1673,15 @@ extern "C" int wf_seq_run_part(wf_seq_engine* e, int layer, int part, int nseq, 
     float* result = e->y;
     const bool parallel = e->cfg.block_form == WF_SEQ_BLOCK_PARALLEL;
     const bool post = e->cfg.block_form == WF_SEQ_BLOCK_POST || parallel;
-    if (part == 5 && !(parallel && L.c.has_ff && !e->cfg.one_norm)) { set_error("wf_seq_run_part: layer %d has no second norm", layer); return WF_ERR_INVALID; }
-    if (post && (part == 1 || part == 4)) { set_error("wf_seq_run_part: this model's sublayers have no input convolution"); return WF_ERR_INVALID; }
-    if (part == 0 && e->cfg.layer_norm) {
+    const bool dyn = e->cfg.norm_kind == WF_SEQ_NORM_DYN_TANH;
+    if (part == 5 && !(L.c.has_ff && (dyn || (parallel && !e->cfg.one_norm)))) { set_error("wf_seq_run_part: layer %d has no second norm", layer); return WF_ERR_INVALID; }
+    if (part >= 6 && !(dyn && (part == 6 || (part == 7 && L.c.has_ff)))) { set_error("wf_seq_run_part: layer %d has no norm behind that sublayer", layer); return WF_ERR_INVALID; }
+    if ((post || dyn) && (part == 1 || part == 4)) { set_error("wf_seq_run_part: this model's sublayers have no input convolution"); return WF_ERR_INVALID; }
+    if (dyn && (part == 0 || part >= 5)) {
+        if (cuda_check(cudaMemcpyAsync(e->x, in_host, bytes, cudaMemcpyHostToDevice, s), "in")) return WF_ERR_CUDA;
+        rc = launch_dyn_tanh(e->dt, e->x, W, part == 0 ? L.dn1 : part == 5 ? L.dn2 : part == 6 ? L.dn1b : L.dn2b, n, W, e->hn, nullptr, nullptr, s);
+        result = e->hn;
+    } else if (part == 0 && e->cfg.layer_norm) {
         if (cuda_check(cudaMemcpyAsync(e->x, in_host, bytes, cudaMemcpyHostToDevice, s), "in")) return WF_ERR_CUDA;
         rc = launch_layer_norm(e->dt, e->x, W, L.norm1, L.norm1_bias, e->cfg.eps, n, W, e->hn, W, nullptr, 0, nullptr, s);
         result = e->hn;
@@ -1554,7 +1715,7 @@ extern "C" int wf_seq_run_part(wf_seq_engine* e, int layer, int part, int nseq, 
         if (post && cuda_check(cudaMemcpyAsync(e->x, e->hn, bytes, cudaMemcpyDeviceToDevice, s), "in")) return WF_ERR_CUDA;
         rc = launch_gate_mul(e->dt, e->hn, W, e->hn, W, 2, n, W, e->h_t, W, s);
         if (!rc) rc = part == 2 ? run_mixer(e, L, v.b) : run_ff(e, L, v.b);
-        if (!rc && part == 2 && L.ob && post && !parallel && !e->cfg.norm_weights && !L.c.pair) rc = launch_add_bias(e->dt, e->y, W, L.ob, n, W, s);
+        if (!rc && part == 2 && L.ob && norm_takes_bias(e, L)) rc = launch_add_bias(e->dt, e->y, W, L.ob, n, W, s);
     } else { set_error("wf_seq_run_part: unknown part %d", part); return WF_ERR_INVALID; }
     if (rc) return rc;
     if (cuda_check(cudaMemcpyAsync(out_host, result, bytes, cudaMemcpyDeviceToHost, s), "out")) return WF_ERR_CUDA;

@@ -83,8 +83,9 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(GemmArgs g) {
             const int n = tile_n * BN + tx * 4 + j;
             if (n >= g.N) continue;
             const size_t off = (size_t)z * g.sC + (size_t)m * g.ldc + n;
-            if (CF32) ((float*)g.C)[off] = acc[i][j];
-            else ((T*)g.C)[off] = from_f<T>(acc[i][j]);
+            const float v = epilogue_f(g.ep, acc[i][j]);
+            if (CF32) ((float*)g.C)[off] = v;
+            else ((T*)g.C)[off] = from_f<T>(v);
         }
     }
 }
@@ -205,7 +206,7 @@ __global__ void __launch_bounds__(128) gemm_mma_kernel(GemmArgs g) {
                     const int n = tile_n * BN + wn * 32 + j * 8 + c + e;
                     if (n >= g.N) continue;
                     const size_t off = (size_t)z * g.sC + (size_t)m * g.ldc + n;
-                    const float v = acc[i][j][h * 2 + e];
+                    const float v = epilogue_f(g.ep, acc[i][j][h * 2 + e]);
                     if (CF32) ((float*)g.C)[off] = v;
                     else ((__nv_bfloat16*)g.C)[off] = __float2bfloat16_rn(v);
                 }
@@ -293,6 +294,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_rows_kernel(GemmArgs g, Pa
             for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
             if (lane == 0 && m < rows && n0 + r < g.N) {
                 const size_t off = (size_t)(c_row0 + m) * g.ldc + n0 + r;
+                v = epilogue_f(g.ep, v);
                 if (CF32) ((float*)g.C)[off] = v; else ((T*)g.C)[off] = from_f<T>(v);
             }
         }

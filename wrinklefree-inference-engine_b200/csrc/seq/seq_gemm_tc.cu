@@ -35,7 +35,7 @@ constexpr uint32_t TC_SPIN_LIMIT = 1u << 24;
 struct TcParams {
     int M, N, K;
     int n_tiles, tiles;
-    void* C; int ldc, c_f32;
+    void* C; int ldc, c_f32, ep;
     const int32_t* tile_group;     // per 128-token tile: expert, or < 0 = skip (null: dense)
     int group_w_rows;              // weight rows between consecutive experts in the stacked tensor
     int* err;
@@ -197,6 +197,10 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tc_kernel(const __grid_con
                 }
                 const int m0 = mt * TC_TOK + c * 32;
                 const int mcnt = p.M - m0 < 32 ? p.M - m0 : 32;            // warp-uniform
+                if (p.ep != EP_NONE) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(epilogue_f(p.ep, __uint_as_float(r[j])));
+                }
                 if (n_ok) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
@@ -283,7 +287,7 @@ int launch_gemm_tc(const GemmArgs& g, int n_groups, cudaStream_t s) {
     p.M = g.M; p.N = g.N; p.K = g.K;
     p.n_tiles = (g.N + TC_ROWS - 1) / TC_ROWS;
     p.tiles = p.n_tiles * ((g.M + TC_TOK - 1) / TC_TOK);
-    p.C = g.C; p.ldc = g.ldc; p.c_f32 = g.c_f32;
+    p.C = g.C; p.ldc = g.ldc; p.c_f32 = g.c_f32; p.ep = g.ep;
     p.tile_group = g.tile_group; p.group_w_rows = group_w_rows;
     p.err = g_err_dev[dev];
     const int sms = sm_count();

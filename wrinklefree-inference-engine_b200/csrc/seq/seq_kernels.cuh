@@ -42,6 +42,30 @@ struct BranchSum {
     const void *gb1 = nullptr, *gb2 = nullptr;
 };
 int launch_branch_add_norm(int dt, float* x, const BranchSum& bs, const void* w, const void* b, float w_offset, float eps, int n, int W, void* h, cudaStream_t s);
+// Element-wise norm tanh(alpha x) w + b (w, b: T [W]; alpha: T [1]) of the rows of x (float [n, W], row stride ldx; rows: optional gather) as
+// float (y, dense) and / or T (y_t, dense)
+struct DynNorm { const void *w = nullptr, *b = nullptr, *alpha = nullptr; };
+int launch_dyn_tanh(int dt, const float* x, int ldx, const DynNorm& nm, int n, int W, float* y, void* y_t, const int32_t* rows, cudaStream_t s);
+// Everything between two sublayers of a stack with element-wise norms, in one kernel (thread per token and few channels):
+//   v = x (0 with init);  v += post(y + bias) when there is a sublayer output;  v += embed_scale * embed[tokens[i], :] when embed is given;
+//   x = v;  h = pre(v) as T and, where hf is given, as float (pre.w null: neither).
+// The sublayer output is y (float [n, W]) or, with yexp given, the routed experts' combination sum_k wts[i, k] yexp[row(i, k), :] (+ shared_y
+// [i, :]), row(i, k) = pair_row[i * top + k], or i * top + k without pair_row.  x, y, shared_y, h, hf dense.
+struct StreamStep {
+    int init = 0;
+    const float* y = nullptr;
+    const void* bias = nullptr;
+    const float *yexp = nullptr, *wts = nullptr, *shared_y = nullptr;
+    const int32_t* pair_row = nullptr;
+    int top = 0;
+    DynNorm post, pre;
+    const void* embed = nullptr;
+    const int32_t* tokens = nullptr;
+    float embed_scale = 1.f;
+    void* h = nullptr;
+    float* hf = nullptr;
+};
+int launch_stream_step(int dt, float* x, const StreamStep& st, int n, int W, cudaStream_t s);
 // z <- cap * tanh(z / cap) over count floats
 int launch_softcap(float* z, size_t count, float cap, cudaStream_t s);
 // x[i, :] = table[tokens[i], :] + sinusoidal position vector of tok_pos[i] (entry 2k sin, 2k + 1 cos of pos * base^(-2k / W)); x_t: optional T copy
@@ -72,7 +96,9 @@ int launch_norm_taps_rows(int dt, const Batch& b, const float* x, int ldx, const
 int launch_norm_taps(int dt, const Batch& b, const float* x, int ldx, const void* nw, int groups, float eps, const void* cw, int taps, int W, float* state,
                      size_t slot_stride, void* out_t, int ld_t, float* hn, cudaStream_t s);
 
-// C[m, n] = sum_k A[m, k] * B[n, k]  (B stored [N, K] row-major, i.e. a Linear weight), float accumulation.
+// what a product does to its results before it stores them: relu(v)^2, or v (1 + erf(v / sqrt 2)) / 2 (the ungated feed-forward activations)
+enum { EP_NONE = 0, EP_RELU2 = 1, EP_GELU_ERF = 2 };
+// C[m, n] = ep(sum_k A[m, k] * B[n, k])  (B stored [N, K] row-major, i.e. a Linear weight), float accumulation.
 struct GemmArgs {
     const void* A = nullptr; int a_f32 = 0;  // A is T, or float when a_f32 (rounded to T on the tensor-core path)
     int lda = 0;
@@ -88,6 +114,7 @@ struct GemmArgs {
     long long group_stride = 0;
     const int32_t* a_rows = nullptr;
     int n_groups = 1;                        // weight matrices stacked behind B (grouped form)
+    int ep = EP_NONE;
     int algo = 0;                            // 0 = choose; 1 plain FMA, 2 mma.sync, 3 tcgen05, 4 few-row streaming (tests and measurements)
 };
 constexpr int GEMM_BM = 128;                 // row granule of the grouped form (the token tile of the tcgen05 kernel)
@@ -151,6 +178,9 @@ struct GqaDims {
     int chunk = 0, sink = 0, gate_elem = 0; float softcap = 0.f;
     const float* rel = nullptr; int rel_n = 0;
     int v_is_k = 0;               // the values are the cached keys (dv == d): a page holds keys only, nothing is projected or stored for values
+    int keep_first = 0;           // positions below it stay visible however far the window has moved on
+    // rotation: the pairs' frequencies (device, double [rope_dims / 2]; null: rope_base^(-2i / rope_dims)), the factor on cosines and sines
+    const double* freq = nullptr; float mscale = 1.f;
     // dist_r1 / dist_r2 (float [H], device): score -= r1[h] ln(1 + r2[h] (i - j)).  sink_h (float [H], device; sink = 2): the denominator carries
     // exp(sink_h[h]).  talk (float [H, H], device): the heads' weights are mixed before the value sum, w_h <- sum_g talk[h, g] w_g.
     const float *dist_r1 = nullptr, *dist_r2 = nullptr, *sink_h = nullptr, *talk = nullptr;
@@ -163,8 +193,8 @@ long long gqa_cache_elems(const GqaDims& D, int page_size);
 // = sigmoid of the gate logits (1 when g_off < 0; gate null: not written); [n, H * dv] with D.gate_elem.
 int launch_gqa_prep(int dt, const Batch& b, const GqaDims& D, const float* proj, int ld, int k_off, int v_off, int g_off, const void* qb, const void* kb,
                     const void* vb, float eps, const PagedCache& pc, void* qn, float* gate, cudaStream_t s);
-// out T [n, H * dv]: per (token, head) softmax over keys j in (pos - window, pos] of q . k_j * scale - slope_h * (pos - j), weighted value
-// sum, times gate[n, H] (null: no gate).
+// out T [n, H * dv]: per (token, head) softmax over keys j in (pos - window, pos] (and j < keep_first) of q . k_j * scale - slope_h * (pos - j),
+// weighted value sum, times gate[n, H] (null: no gate).
 int launch_gqa_attn(int dt, const Batch& b, const GqaDims& D, const void* qn, const float* gate, const PagedCache& pc, void* out, cudaStream_t s);
 
 // Attention whose heads' weights are mixed (D.talk) has kernels of its own: a plain one behind launch_gqa_attn, and tensor-core forms
@@ -241,7 +271,8 @@ struct RouterDims {
     int norm = 0;                  // 1: weights divided by the sum of the chosen scores (+ 1e-20)
     float scale = 1.f;             // weights multiplied by this
 };
-// z float [n, E + I] (ldz) -> ids [n, top], wts [n, top]; counts[E] += tokens per real expert (zero on entry; null: not counted)
+// z float [n, E + I] (ldz) -> ids [n, top], wts [n, top]; counts[E] += tokens per real expert (zero on entry; null: not counted);
+// correction: T [E + I] added to the scores for the choice only (null: nothing)
 int launch_moe_route(int dt, const RouterDims& R, int n, const float* z, int ldz, const void* correction, int32_t* ids, float* wts,
                      int32_t* counts, cudaStream_t s);
 // the router product and the choice in one kernel: z[i, 0..NZ) = w[NZ, W] . x[i, :] with x FLOAT (ldx) and float products, then the choice

@@ -28,7 +28,7 @@ __device__ void route_token(const RouterDims& R, const float* zr, const T* __res
     float* ch = sc + N;
     float* gs = ch + N;
     if (R.act == 1) {
-        for (int e = lane; e < N; e += 32) { sc[e] = sigmoid_f(zr[e]); ch[e] = sc[e] + to_f(correction[e]); }
+        for (int e = lane; e < N; e += 32) { sc[e] = sigmoid_f(zr[e]); ch[e] = sc[e] + (correction ? to_f(correction[e]) : 0.f); }
     } else {
         float mx = -INFINITY;
         for (int e = lane; e < N; e += 32) mx = fmaxf(mx, zr[e]);
@@ -37,7 +37,7 @@ __device__ void route_token(const RouterDims& R, const float* zr, const T* __res
         for (int e = lane; e < N; e += 32) { const float p = expf(zr[e] - mx); sc[e] = p; sum += p; }
         sum = warp_sum(sum);
         const float inv = 1.f / sum;
-        for (int e = lane; e < N; e += 32) { sc[e] *= inv; ch[e] = sc[e] + to_f(correction[e]); }
+        for (int e = lane; e < N; e += 32) { sc[e] *= inv; ch[e] = sc[e] + (correction ? to_f(correction[e]) : 0.f); }
     }
     __syncwarp();
     // group score = sum of the group's group_top largest choice scores (the largest alone when group_top <= 1); keep the best `keep` groups

@@ -1,4 +1,5 @@
-// Row-wise kernels of the sequence models: embedding gather, grouped RMS norm (+ residual add), causal depthwise taps with carried state.
+// Row-wise kernels of the sequence models: embedding gather, grouped RMS norm (+ residual add), element-wise norms with everything that lies
+// between two sublayers, causal depthwise taps with carried state.
 #include "seq_kernels.cuh"
 
 namespace wf {
@@ -435,6 +436,114 @@ int launch_branch_add_norm(int dt, float* x, const BranchSum& bs, const void* w,
     if (dt == WF_BF16) branch_add_norm_kernel<<<n, row_threads(W), 0, s>>>(x, bs, (const __nv_bfloat16*)w, (const __nv_bfloat16*)b, w_offset, eps, W, (__nv_bfloat16*)h);
     else branch_add_norm_kernel<<<n, row_threads(W), 0, s>>>(x, bs, (const float*)w, (const float*)b, w_offset, eps, W, (float*)h);
     return launch_check(cudaGetLastError(), "branch_add_norm");
+}
+
+// ---- element-wise norms (tanh(alpha x) w + b): no row statistics, so everything between two sublayers is one pass over the row ----------
+template <typename T>
+__global__ void dyn_tanh_kernel(const float* __restrict__ x, int ldx, const T* __restrict__ w, const T* __restrict__ b, const T* __restrict__ alpha, int W,
+                                float* __restrict__ y, T* __restrict__ y_t, const int32_t* __restrict__ rows) {
+    const int i = blockIdx.x;
+    const float* xr = x + (size_t)(rows ? rows[i] : i) * ldx;
+    const float al = to_f(alpha[0]);
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += gridDim.y * blockDim.x) {
+        const float v = fmaf(tanhf(al * xr[c]), to_f(w[c]), to_f(b[c]));
+        if (y) y[(size_t)i * W + c] = v;
+        if (y_t) y_t[(size_t)i * W + c] = from_f<T>(v);
+    }
+}
+
+int launch_dyn_tanh(int dt, const float* x, int ldx, const DynNorm& nm, int n, int W, float* y, void* y_t, const int32_t* rows, cudaStream_t s) {
+    if (n <= 0) return WF_OK;
+    if (!nm.w || !nm.b || !nm.alpha) { set_error("dyn_tanh: weight, bias and alpha are needed"); return WF_ERR_INVALID; }
+    const dim3 grid(n, n < 256 ? (W + 255) / 256 : 1);
+    if (dt == WF_BF16) dyn_tanh_kernel<<<grid, 256, 0, s>>>(x, ldx, (const __nv_bfloat16*)nm.w, (const __nv_bfloat16*)nm.b, (const __nv_bfloat16*)nm.alpha, W, y, (__nv_bfloat16*)y_t, rows);
+    else dyn_tanh_kernel<<<grid, 256, 0, s>>>(x, ldx, (const float*)nm.w, (const float*)nm.b, (const float*)nm.alpha, W, y, (float*)y_t, rows);
+    return launch_check(cudaGetLastError(), "dyn_tanh");
+}
+
+template <typename T> __device__ __forceinline__ void load_n(const T* p, float (&v)[1]) { v[0] = to_f(p[0]); }
+template <typename T> __device__ __forceinline__ void load_n(const T* p, float (&v)[4]) { const float4 q = load4(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+template <typename T> __device__ __forceinline__ void store_n(T* p, const float (&v)[1]) { p[0] = from_f<T>(v[0]); }
+template <typename T> __device__ __forceinline__ void store_n(T* p, const float (&v)[4]) { store4(p, v); }
+
+// v += / = tanh(alpha u) w + b for VEC channels at c
+template <typename T, int VEC>
+__device__ __forceinline__ void dyn_apply(const DynNorm& nm, int c, const float (&u)[VEC], float (&out)[VEC]) {
+    float w[VEC], b[VEC];
+    load_n((const T*)nm.w + c, w);
+    load_n((const T*)nm.b + c, b);
+    const float al = to_f(((const T*)nm.alpha)[0]);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) out[e] = fmaf(tanhf(al * u[e]), w[e], b[e]);
+}
+
+// grid (tokens, channel blocks).  VEC = 4: W a multiple of 4 (rows 16-byte aligned)
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) stream_step_kernel(float* __restrict__ x, StreamStep st, int W) {
+    const int i = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
+    if (c >= W) return;
+    const size_t at = (size_t)i * W + c;
+    float v[VEC];
+    if (st.init) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = 0.f;
+    } else load_n(x + at, v);
+    if (st.y || st.yexp) {
+        float u[VEC], d[VEC];
+        if (st.yexp) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) u[e] = 0.f;
+            for (int k = 0; k < st.top; ++k) {
+                const size_t pi = (size_t)i * st.top + k;
+                const float w = st.wts[pi];
+                float q[VEC];
+                load_n(st.yexp + (st.pair_row ? (size_t)st.pair_row[pi] : pi) * W + c, q);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) u[e] = fmaf(w, q[e], u[e]);
+            }
+            if (st.shared_y) {
+                float q[VEC];
+                load_n(st.shared_y + at, q);
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) u[e] += q[e];
+            }
+        } else load_n(st.y + at, u);
+        if (st.bias) {
+            float q[VEC];
+            load_n((const T*)st.bias + c, q);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) u[e] += q[e];
+        }
+        dyn_apply<T, VEC>(st.post, c, u, d);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] += d[e];
+    }
+    if (st.embed) {
+        float q[VEC];
+        load_n((const T*)st.embed + (size_t)st.tokens[i] * W + c, q);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = fmaf(st.embed_scale, q[e], v[e]);
+    }
+    store_n(x + at, v);
+    if (st.pre.w) {
+        float h[VEC];
+        dyn_apply<T, VEC>(st.pre, c, v, h);
+        store_n((T*)st.h + at, h);
+        if (st.hf) store_n(st.hf + at, h);
+    }
+}
+
+int launch_stream_step(int dt, float* x, const StreamStep& st, int n, int W, cudaStream_t s) {
+    if (n <= 0) return WF_OK;
+    if (((st.y || st.yexp) && !st.post.w) || (st.y && st.yexp) || (st.yexp && (!st.wts || st.top < 1)) || (st.embed && !st.tokens) || (st.pre.w && !st.h)) {
+        set_error("stream_step: inconsistent inputs"); return WF_ERR_INVALID;
+    }
+    const int vec = W % 4 == 0 ? 4 : 1, per = W / vec;
+    const int threads = per >= 256 && n >= sm_count() ? 256 : (per > 64 ? 128 : 64);      // few tokens: more, smaller blocks
+    const dim3 grid(n, (per + threads - 1) / threads);
+    if (dt == WF_BF16) { if (vec == 4) stream_step_kernel<__nv_bfloat16, 4><<<grid, threads, 0, s>>>(x, st, W); else stream_step_kernel<__nv_bfloat16, 1><<<grid, threads, 0, s>>>(x, st, W); }
+    else { if (vec == 4) stream_step_kernel<float, 4><<<grid, threads, 0, s>>>(x, st, W); else stream_step_kernel<float, 1><<<grid, threads, 0, s>>>(x, st, W); }
+    return launch_check(cudaGetLastError(), "stream_step");
 }
 
 __global__ void softcap_kernel(float* __restrict__ z, size_t count, float cap) {

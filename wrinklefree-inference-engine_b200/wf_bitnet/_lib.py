@@ -115,7 +115,8 @@ WF_SEQ_F32, WF_SEQ_BF16 = 0, 1
 WF_SEQ_LATENT_ATTENTION, WF_SEQ_DELTA, WF_SEQ_GQA_ATTENTION, WF_SEQ_SSD, WF_SEQ_MINGRU, WF_SEQ_MLSTM, WF_SEQ_GLA = 0, 1, 2, 3, 4, 5, 6
 WF_SEQ_BLOCK_SANDWICH, WF_SEQ_BLOCK_POST, WF_SEQ_BLOCK_PARALLEL = 0, 1, 2
 WF_SEQ_FF_NONE, WF_SEQ_FF_ROUTED, WF_SEQ_FF_DENSE = 0, 1, 2
-WF_SEQ_ACT_SILU, WF_SEQ_ACT_CLAMPED, WF_SEQ_ACT_GELU_TANH, WF_SEQ_ACT_RELU2 = 0, 1, 2, 3
+WF_SEQ_ACT_SILU, WF_SEQ_ACT_CLAMPED, WF_SEQ_ACT_GELU_TANH, WF_SEQ_ACT_RELU2, WF_SEQ_ACT_GELU_ERF = 0, 1, 2, 3, 4
+WF_SEQ_NORM_RMS, WF_SEQ_NORM_DYN_TANH = 0, 1
 WF_SEQ_QKNORM_NONE, WF_SEQ_QKNORM_UNIT, WF_SEQ_QKNORM_HEAD, WF_SEQ_QKNORM_FULL = 0, 1, 2, 3
 
 
@@ -141,6 +142,7 @@ class SeqLayer(C.Structure):
         ("rope_factor", C.c_float), ("rope_orig", C.c_float), ("rope_fast", C.c_float), ("rope_slow", C.c_float),
         ("v_is_k", C.c_int), ("gate_cap", C.c_float),
         ("dist_log", C.c_int), ("talk", C.c_int), ("pair_norm", C.c_int), ("decay_tau", C.c_float),
+        ("keep_first", C.c_int), ("no_correction", C.c_int), ("shared_plain", C.c_int),
     ]
 
     def __init__(self, *a, **kw):
@@ -160,6 +162,7 @@ class SeqConfig(C.Structure):
         ("n_extra", C.c_int), ("embed_scale", C.c_float), ("norm_weights", C.c_int), ("tied_head", C.c_int),
         ("norm_offset", C.c_float),
         ("layer_norm", C.c_int), ("one_norm", C.c_int), ("branch_gates", C.c_int), ("max_positions", C.c_int), ("logit_softcap", C.c_float),
+        ("norm_kind", C.c_int), ("loop_start", C.c_int), ("loop_stop", C.c_int), ("loop_times", C.c_int),
     ]
 
 
@@ -170,6 +173,7 @@ SEQ_SYMBOLS = {
     "wf_seq_create": (_i, [C.POINTER(SeqConfig), C.POINTER(SeqLayer), C.POINTER(_vp)]),
     "wf_seq_destroy": (None, [_vp]),
     "wf_seq_device_bytes": (_sz, [_vp]),
+    "wf_seq_layer_runs": (_i, [_vp]),
     "wf_seq_set_tensor": (_i, [_vp, C.c_char_p, _vp, _sz, _i]),
     "wf_seq_tensor_count": (_i, [_vp]),
     "wf_seq_tensor_name": (C.c_char_p, [_vp, _i, C.POINTER(_sz), C.POINTER(_i)]),

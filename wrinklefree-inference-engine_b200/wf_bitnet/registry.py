@@ -23,6 +23,8 @@ _MODULES: Dict[str, str] = {
     "FivedraForCausalLM": "sglang.srt.models.fivedra",
     "Fuvavik": "sglang.srt.models.fuvavik",
     "FuvavikForCausalLM": "sglang.srt.models.fuvavik",
+    "Kilizen": "sglang.srt.models.kilizen",
+    "KilizenForCausalLM": "sglang.srt.models.kilizen",
 }
 
 

@@ -61,6 +61,10 @@ class SeqEngine:
     def finalize(self) -> None:
         seq_check(seq_lib().wf_seq_finalize(self._h))
 
+    def layer_runs(self) -> int:
+        """Layers a token passes: a layer inside the configuration's loop counts once per pass."""
+        return int(seq_lib().wf_seq_layer_runs(self._h))
+
     def device_bytes(self) -> int:
         return int(seq_lib().wf_seq_device_bytes(self._h))
 
@@ -105,7 +109,7 @@ class SeqEngine:
     # ---- parity taps / measurement
     def step_with_layer_tap(self, slots, counts, tokens, want=()):
         n = int(np.sum(counts))
-        tap = np.empty((self.cfg.n_layers, n, self.width), dtype=np.float32)
+        tap = np.empty((self.layer_runs(), n, self.width), dtype=np.float32)
         seq_check(seq_lib().wf_seq_set_layer_tap(self._h, tap.ctypes.data))
         try:
             out = self.step(slots, counts, tokens, want)
