@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """bench.py — decode throughput of the BitNet-2B-4T-shaped hot path on B200.
 
-    python bench.py --gpus N --steps K --warmup W [--impl reference] [--workload bs64|bs1|hybrid|tutizen|nukezen|fivedra|fuvavik]
+    python bench.py --gpus N --steps K --warmup W [--impl reference] [--workload bs64|bs1|hybrid|tutizen|nukezen|fivedra|fuvavik|kilizen]
 
 --workload hybrid (1 GPU) measures the layer-stack sequence engine (latent attention / gated delta rule / routed feed-forward) instead:
 prefill and decode tok/s at two layer sizes with random weights, per launch-group times, and the BitNet engine at equal size beside it.
@@ -1194,23 +1194,87 @@ def run_fuvavik(args):
     return 0
 
 
+# --workload kilizen: the Kilizen design (element-wise tanh norms around every sublayer; window attention with kept first positions whose values
+# are the projected keys, run twice by a loop; a matrix memory; causal attention with biases and a norm over the whole projection; learned
+# sinks; ungated units dense / routed with a plain shared expert) on the sequence engine at sizes that resemble real layers, random weights,
+# beside the closest existing models on the same engine at equal width / heads / layers: Tutizen (grouped-query attention, routed with a
+# shared expert, equal experts) and, for the matrix memory, Fivedra's paired layers.
+KILIZEN_SIZES = {
+    "w1024": dict(rot=64, keep=4, mem=dict(heads=8, d=64, dv=128)),
+    "w2560": dict(rot=64, keep=4, mem=dict(heads=20, d=128, dv=128)),
+}
+
+
+def kilizen_config(z, f, window):
+    """z: the Tutizen size of the same name (width, heads, experts, vocabulary), f: what only this design has"""
+    g = f["mem"]
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "shared": {"ff": z["ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["d"], "vdim": z["dv"], "scale": z["d"] ** -0.5}
+    win = dict(att, mask={"size": window, "keep_first": f["keep"]},
+               rot={"dims": f["rot"], "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    layers = [{"type": "attention", "mixer": win, "mlp": moe},
+              {"type": "mlstm", "mixer": {"heads": g["heads"], "dim": g["d"], "vdim": g["dv"], "gate_cap": 15.0}, "mlp": moe},
+              {"type": "attention_2", "mixer": dict(att, rot={"dims": z["d"], "base": 10000.0}), "mlp": {"kind": "dense", "ff": z["top"] * z["ff"]}}]
+    return {"architecture": "Kilizen", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "loop": {"start": 0, "stop": 1, "times": 2}, "layers": layers}
+
+
+def run_kilizen(args):
+    from wf_bitnet import _lib
+    torch.cuda.set_device(0)
+    _lib.require_gpu()
+    K, W_ = max(2, args.steps), max(3, args.warmup)
+    peak, peak_src = measured_peaks()
+    sampler = ClockSampler(0)
+    sampler.start()
+    out, launches = {}, 0
+    for name, f in KILIZEN_SIZES.items():
+        if args.hybrid_size and name != args.hybrid_size:
+            continue
+        z, window = TUTIZEN_SIZES[name], NUKEZEN_SIZES[name]["window"]
+        prompt = 2048
+        decode_points = [(1, 512), (8, 2048), (64, 4096)] if name == "w2560" else [(1, 512), (8, 1024), (64, 1024)]
+        cfg = kilizen_config(z, f, window)
+        res, n1 = measure_seq_model(cfg, prompt, decode_points, K)
+        res["layer_runs"] = ["attention + moe", "attention + moe (second pass)", "mlstm + moe", "attention_2 + dense"]
+        g = f["mem"]
+        # state one decoded token reads and writes per matrix-memory layer (float); cached bytes per attention layer and 1000 tokens of context
+        res["state_bytes"] = 4 * g["heads"] * (g["d"] * (g["dv"] + 1) + 1)
+        res["kv_bytes_per_layer_per_1k_ctx"] = 1000 * z["kv_heads"] * (z["d"] + z["dv"]) * 2
+        tres, n2 = measure_seq_model(tutizen_config(z), prompt, decode_points, K)
+        res["tutizen_equal_size"] = tres
+        fcfg, fshapes = fivedra_config(NUKEZEN_SIZES[name], FIVEDRA_SIZES[name], paired_only=True)
+        fres, n3 = measure_seq_model(fcfg, prompt, decode_points, K, fshapes)
+        res["fivedra_paired_equal_size"] = fres
+        launches += n1 + n2 + n3
+        out[name] = res
+    clocks = sampler.stop()
+    head = out.get("w2560") or next(iter(out.values()))
+    top = sorted(head["decode"].items())[-1]
+    emit({"metric": "prefill / decode tok/s of the Kilizen design on the sequence engine beside Tutizen at equal size", "workload": "kilizen",
+          "value": top[1]["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W_, "higher_is_better": True, "dtype": "bf16",
+          "data": "synthetic (random weights; decode contexts are whatever the cache pages hold)", "vs_baseline": None,
+          "config": {"model": "Kilizen-shaped, " + ", ".join(out), "point": top[0], "l2": "weights per step exceed L2 (126 MB) at w2560; w1024 is L2-resident"},
+          "hbm_peak_gbs": peak, "peak_source": peak_src, "sizes": out, "clocks": clocks, "gpu_launches": launches})
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="bs64", choices=["bs64", "bs1", "hybrid", "tutizen", "nukezen", "fivedra", "fuvavik"] + sorted(TP_WORKLOADS))
-    ap.add_argument("--hybrid-size", default="", help="--workload hybrid / tutizen / nukezen / fivedra / fuvavik: run only this size (w1024 | w2560)")
+    ap.add_argument("--workload", default="bs64", choices=["bs64", "bs1", "hybrid", "tutizen", "nukezen", "fivedra", "fuvavik", "kilizen"] + sorted(TP_WORKLOADS))
+    ap.add_argument("--hybrid-size", default="", help="--workload hybrid / tutizen / nukezen / fivedra / fuvavik / kilizen: run only this size (w1024 | w2560)")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--no-aux", action="store_true", help="skip the batch-1 aux measurement")
     ap.add_argument("--no-tp", action="store_true", help="skip the tensor-parallel suite (aux.tp)")
     args = ap.parse_args()
-    if args.workload in ("hybrid", "tutizen", "nukezen", "fivedra", "fuvavik"):
+    if args.workload in ("hybrid", "tutizen", "nukezen", "fivedra", "fuvavik", "kilizen"):
         if args.impl == "reference":
             emit({"impl": "reference", "unavailable": "the reference has no model of this design; its arm is defined for the 2B workloads only"})
             return 0
-        return {"hybrid": run_hybrid, "tutizen": run_tutizen, "nukezen": run_nukezen, "fivedra": run_fivedra, "fuvavik": run_fuvavik}[args.workload](args)
+        return {"hybrid": run_hybrid, "tutizen": run_tutizen, "nukezen": run_nukezen, "fivedra": run_fivedra, "fuvavik": run_fuvavik, "kilizen": run_kilizen}[args.workload](args)
     if args.workload in TP_WORKLOADS:
         if args.impl == "reference":
             emit({"impl": "reference", "unavailable": "the reference arm is defined for the 2B workloads (bs64 / bs1) only"})

@@ -21,20 +21,21 @@ constexpr int GA_WARPS = 4;
 constexpr int GA_MAXD = 16;    // per-head sizes up to 32 * 16
 
 constexpr int GA_MAXROT = 256;  // rotated pairs per head
+constexpr int GP_MAXW = 16;     // most warps of a gqa_prep_kernel block
 
-// One block per token; its warps walk the token's head vectors (H query heads, then G key heads, then G value heads): bias, norm
+// One block per token (of 4 warps, or of 16 when the tokens are few and the walk's length counts); its warps walk the token's head vectors (H query heads, then G key heads, then G value heads): bias, norm
 // (per head, or over the whole projection with two block-wide sums first), rotation, store.  The cosines and sines of the token's
 // angles are formed once per block in double, so that the float values are the correctly rounded ones at any position.
 // MAXD: values a lane holds of one head vector (head sizes up to 32 * MAXD).
 template <typename T, int MAXD>
-__global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDims D, const float* __restrict__ proj, int ld, int k_off, int v_off, int g_off,
+__global__ void __launch_bounds__(GP_MAXW * 32) gqa_prep_kernel(Batch b, GqaDims D, const float* __restrict__ proj, int ld, int k_off, int v_off, int g_off,
                                                                    const T* __restrict__ qb, const T* __restrict__ kb, const T* __restrict__ vb, float eps,
                                                                    PagedCache pc, T* __restrict__ qn, float* __restrict__ gate) {
     __shared__ float rot_c[GA_MAXROT], rot_s[GA_MAXROT];
-    __shared__ float vec[GA_WARPS][32 * MAXD];
+    extern __shared__ float vec[];                        // [warps][32 * MAXD]
     __shared__ float scratch[33];
     const int i = blockIdx.x;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const int sq = b.tok_seq[i], pos = b.tok_pos[i];
     const float* row = proj + (size_t)i * ld;
     const int units = D.H + (k_off >= 0 ? (D.v_is_k ? D.G : 2 * D.G) : 0);      // the values are stored only when they are not the keys
@@ -49,7 +50,9 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
         const double lb = log2((double)D.rope_base);
         for (int p = threadIdx.x; p < half; p += blockDim.x) {
             const double a = (double)pos * (D.freq ? D.freq[p] : exp2(-2.0 * (double)p / (double)D.rope_dims * lb));
-            rot_c[p] = (float)cos(a) * D.mscale; rot_s[p] = (float)sin(a) * D.mscale;
+            double sn, cs;
+            sincos(a, &sn, &cs);
+            rot_c[p] = (float)cs * D.mscale; rot_s[p] = (float)sn * D.mscale;
         }
     }
     float inv_q = 1.f, inv_k = 1.f;
@@ -67,7 +70,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
     __syncthreads();
     const T* qw = (const T*)D.q_norm_w;
     const T* kw = (const T*)D.k_norm_w;
-    for (int u = warp; u < units; u += GA_WARPS) {
+    for (int u = warp; u < units; u += nw) {
         const float* src; const T* bias; T* dst; int dim; int norm; const T* nw = nullptr; float inv_all = 1.f; bool rot;
         if (u < D.H) {
             src = row + (size_t)u * D.d; bias = qb ? qb + (size_t)u * D.d : nullptr; dst = qn + ((size_t)i * D.H + u) * D.d; dim = D.d; norm = D.qk_norm; rot = half > 0;
@@ -96,7 +99,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) gqa_prep_kernel(Batch b, GqaDim
 #pragma unroll
         for (int t = 0; t < MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) v[t] = v[t] * inv * (nw ? to_f(nw[c]) : 1.f); }
         if (rot) {
-            float* sv = vec[warp];
+            float* sv = vec + warp * 32 * MAXD;
             __syncwarp();
 #pragma unroll
             for (int t = 0; t < MAXD; ++t) { const int c = lane + 32 * t; if (c < dim) sv[c] = v[t]; }
@@ -307,7 +310,8 @@ int launch_gqa_prep(int dt, const Batch& b, const GqaDims& D, const float* proj,
     if (int rc = check_dims(D)) return rc;
     if (!D.v_is_k && (k_off >= 0) != (v_off >= 0)) { set_error("attention: keys and values are projected together or not at all"); return WF_ERR_INVALID; }
     const bool small = D.d <= 128 && D.dv <= 128;
-#define GP_LAUNCH(T, MD) gqa_prep_kernel<T, MD><<<b.n, GA_WARPS * 32, 0, s>>>(b, D, proj, ld, k_off, v_off, g_off, (const T*)qb, (const T*)kb, (const T*)vb, eps, pc, (T*)qn, gate)
+    const int threads = 32 * (b.n <= sm_count() ? GP_MAXW : GA_WARPS);
+#define GP_LAUNCH(T, MD) gqa_prep_kernel<T, MD><<<b.n, threads, (size_t)threads * MD * sizeof(float), s>>>(b, D, proj, ld, k_off, v_off, g_off, (const T*)qb, (const T*)kb, (const T*)vb, eps, pc, (T*)qn, gate)
     if (dt == WF_BF16) { if (small) GP_LAUNCH(__nv_bfloat16, 4); else GP_LAUNCH(__nv_bfloat16, GA_MAXD); }
     else { if (small) GP_LAUNCH(float, 4); else GP_LAUNCH(float, GA_MAXD); }
 #undef GP_LAUNCH

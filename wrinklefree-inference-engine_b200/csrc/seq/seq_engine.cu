@@ -589,7 +589,7 @@ int run_gqa(wf_seq_engine* e, LayerState& L, const Batch& b, float* out) {
         }
         if ((rc = launch_gqa_attn_mma(b, D, e->qn, gate, pc, e->og, e->gqa_ws, splits, s))) return rc;
     } else if ((rc = launch_gqa_attn(e->dt, b, D, e->qn, gate, pc, e->og, s))) return rc;
-    mark(e, D.talk ? "attn.attention(mixed heads)" : D.softcap > 0.f || D.rel ? "attn.attention(cap+bias)" : "attn.attention");
+    mark(e, D.talk ? "attn.attention(mixed heads)" : D.softcap > 0.f || D.rel ? "attn.attention(cap+bias)" : D.keep_first > 0 ? "attn.attention(window+first)" : "attn.attention");
     rc = launch_gemm(e->dt, lin(e->og, 0, nv, L.wo, nv, out, 1, W, n, W, nv), s);
     if (!rc && L.ob && !(norm_takes_bias(e, L) && out == e->y)) rc = launch_add_bias(e->dt, out, W, L.ob, n, W, s);
     mark(e, "attn.out_gemm");

@@ -107,9 +107,10 @@ __global__ void moe_route_kernel(RouterDims R, const float* __restrict__ z, int 
 // and warp t makes the choice of token t from the shared copy.
 // RF_TB bounds tb.  Measured at 2048 tokens x 31 rows x 2560: 8 tokens per block 70 us, 1 token per block 75 us (the weight rows come from
 // L2 either way; fewer, longer blocks fill the machine worse), while single decoded tokens pay for the unused accumulators: so 1.
-constexpr int RF_THREADS = 256, RF_TB = 1;
-template <typename T, bool VEC>
-__global__ void __launch_bounds__(RF_THREADS) router_fused_kernel(RouterDims R, int n, int tb, const float* __restrict__ x, int ldx, const T* __restrict__ w, int NZ, int W,
+// NT: threads of a block — one warp per router row when the tokens do not fill the machine by themselves.
+constexpr int RF_THREADS = 256, RF_THREADS_FEW = 1024, RF_TB = 1;
+template <typename T, bool VEC, int NT>
+__global__ void __launch_bounds__(NT) router_fused_kernel(RouterDims R, int n, int tb, const float* __restrict__ x, int ldx, const T* __restrict__ w, int NZ, int W,
                                                                   float* __restrict__ z, int ldz, const T* __restrict__ correction, int32_t* __restrict__ ids,
                                                                   float* __restrict__ wts, int32_t* __restrict__ counts) {
     extern __shared__ __align__(16) float sm[];
@@ -119,11 +120,11 @@ __global__ void __launch_bounds__(RF_THREADS) router_fused_kernel(RouterDims R, 
     float* scratch = zl + (size_t)tb * NZ;           // [tb][per]: route_token's
     const int i0 = blockIdx.x * tb, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int nt = n - i0 < tb ? n - i0 : tb;
-    if (RF_TB == 1) { for (int c = threadIdx.x; c < W; c += RF_THREADS) xs[c] = x[(size_t)i0 * ldx + c]; }
-    else for (int idx = threadIdx.x; idx < nt * W; idx += RF_THREADS) { const int t = idx / W, c = idx - t * W; xs[(size_t)t * Wp + c] = x[(size_t)(i0 + t) * ldx + c]; }
+    if (RF_TB == 1) { for (int c = threadIdx.x; c < W; c += NT) xs[c] = x[(size_t)i0 * ldx + c]; }
+    else for (int idx = threadIdx.x; idx < nt * W; idx += NT) { const int t = idx / W, c = idx - t * W; xs[(size_t)t * Wp + c] = x[(size_t)(i0 + t) * ldx + c]; }
     __syncthreads();
     constexpr int VN = 16 / sizeof(T);               // elements per 16-byte load
-    for (int e = warp; e < NZ; e += RF_THREADS / 32) {
+    for (int e = warp; e < NZ; e += NT / 32) {
         const T* wr = w + (size_t)e * W;
         float acc[RF_TB];
 #pragma unroll
@@ -297,13 +298,13 @@ int launch_router_fused(int dt, const RouterDims& R, int n, const float* x, int 
     const size_t esz = dt == WF_BF16 ? 2 : 4;
     const bool vec = (W * esz) % 16 == 0 && (((uintptr_t)w) & 15) == 0;
     const int blocks = (n + tb - 1) / tb;
-    if (dt == WF_BF16) {
-        if (vec) router_fused_kernel<__nv_bfloat16, true><<<blocks, RF_THREADS, smem, s>>>(R, n, tb, x, ldx, (const __nv_bfloat16*)w, NZ, W, z, ldz, (const __nv_bfloat16*)correction, ids, wts, counts);
-        else router_fused_kernel<__nv_bfloat16, false><<<blocks, RF_THREADS, smem, s>>>(R, n, tb, x, ldx, (const __nv_bfloat16*)w, NZ, W, z, ldz, (const __nv_bfloat16*)correction, ids, wts, counts);
-    } else {
-        if (vec) router_fused_kernel<float, true><<<blocks, RF_THREADS, smem, s>>>(R, n, tb, x, ldx, (const float*)w, NZ, W, z, ldz, (const float*)correction, ids, wts, counts);
-        else router_fused_kernel<float, false><<<blocks, RF_THREADS, smem, s>>>(R, n, tb, x, ldx, (const float*)w, NZ, W, z, ldz, (const float*)correction, ids, wts, counts);
-    }
+    const bool few = n <= sm_count();
+#define RF_LAUNCH(T, VEC, NT) router_fused_kernel<T, VEC, NT><<<blocks, NT, smem, s>>>(R, n, tb, x, ldx, (const T*)w, NZ, W, z, ldz, (const T*)correction, ids, wts, counts)
+#define RF_PICK(T) do { if (vec) { if (few) RF_LAUNCH(T, true, RF_THREADS_FEW); else RF_LAUNCH(T, true, RF_THREADS); } \
+                        else { if (few) RF_LAUNCH(T, false, RF_THREADS_FEW); else RF_LAUNCH(T, false, RF_THREADS); } } while (0)
+    if (dt == WF_BF16) RF_PICK(__nv_bfloat16); else RF_PICK(float);
+#undef RF_PICK
+#undef RF_LAUNCH
     return launch_check(cudaGetLastError(), "router_fused");
 }
 
